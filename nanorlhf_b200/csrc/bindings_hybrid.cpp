@@ -68,14 +68,16 @@ void act_cols(const Tensor& in, Tensor out, int64_t act) {
         "act_cols");
 }
 
-void gated_part_rmsnorm(const Tensor& y, const Tensor& gate, const Tensor& w, int64_t part, int64_t gate_act, bool gate_first,
+void gated_part_rmsnorm(const Tensor& y, const c10::optional<Tensor>& gate, const Tensor& w, int64_t part, int64_t gate_act, bool gate_first,
                         double eps, double scale, Tensor out) {
   c10::cuda::CUDAGuard guard(out.device());
-  TORCH_CHECK(y.dim() == 2 && gate.dim() == 2 && out.dim() == 2 && gate.size(1) == y.size(1) && out.size(1) == y.size(1) &&
-                  gate.size(0) == y.size(0) && out.size(0) == y.size(0), "gated_part_rmsnorm: shapes");
+  TORCH_CHECK(y.dim() == 2 && out.dim() == 2 && out.size(1) == y.size(1) && out.size(0) == y.size(0), "gated_part_rmsnorm: shapes");
+  if (gate.has_value())
+    TORCH_CHECK(gate->dim() == 2 && gate->size(1) == y.size(1) && gate->size(0) == y.size(0), "gated_part_rmsnorm: gate");
   const bool shared = w.numel() == part;
   TORCH_CHECK(shared || w.numel() == y.size(1), "gated_part_rmsnorm: weight of one part or of all columns");
-  check(nrl_gated_part_rmsnorm(f32(y, "y"), y.stride(0), f32(gate, "gate"), gate.stride(0), f32(w, "w"), shared ? 1 : 0,
+  check(nrl_gated_part_rmsnorm(f32(y, "y"), y.stride(0), gate.has_value() ? f32(*gate, "gate") : nullptr,
+                               gate.has_value() ? gate->stride(0) : 0, f32(w, "w"), shared ? 1 : 0,
                                static_cast<int>(part), static_cast<int>(gate_act), gate_first ? 1 : 0, static_cast<float>(eps),
                                static_cast<float>(scale), out.data_ptr(), out.stride(0), typed(out, "out"),
                                static_cast<int>(y.size(0)), static_cast<int>(y.size(1)), cur_stream()),
@@ -429,7 +431,8 @@ void group_norm_residual(Tensor x, const c10::optional<Tensor>& o, const c10::op
 }
 
 void moe_route(const Tensor& router, const c10::optional<Tensor>& router_bias, int64_t top, const c10::optional<Tensor>& gu, int64_t ff,
-               const c10::optional<Tensor>& act, const c10::optional<Tensor>& ids, const c10::optional<Tensor>& wts) {
+               const c10::optional<Tensor>& act, const c10::optional<Tensor>& ids, const c10::optional<Tensor>& wts, bool sigmoid,
+               bool weight_input) {
   c10::cuda::CUDAGuard guard(router.device());
   TORCH_CHECK(router.dim() == 2, "moe_route: router [T, E]");
   const int T = static_cast<int>(router.size(0)), E = static_cast<int>(router.size(1));
@@ -442,8 +445,8 @@ void moe_route(const Tensor& router, const c10::optional<Tensor>& router_bias, i
   if (wts.has_value()) TORCH_CHECK(ids.has_value() && wts->is_contiguous() && wts->numel() == static_cast<int64_t>(T) * top, "moe_route: wts float [T, top]");
   Tensor wt = wts.has_value() ? *wts : Tensor();
   check(nrl_moe_route(f32(router, "router"), router.stride(0), router_bias.has_value() ? f32(*router_bias, "router_bias") : nullptr, E,
-                      static_cast<int>(top), gu.has_value() ? f32(*gu, "gu") : nullptr, gu.has_value() ? gu->stride(0) : 0,
-                      static_cast<int>(ff), act.has_value() ? act->data_ptr() : nullptr, act.has_value() ? act->stride(0) : 0,
+                      static_cast<int>(top), sigmoid ? 1 : 0, weight_input ? 1 : 0, gu.has_value() ? f32(*gu, "gu") : nullptr,
+                      gu.has_value() ? gu->stride(0) : 0, static_cast<int>(ff), act.has_value() ? act->data_ptr() : nullptr, act.has_value() ? act->stride(0) : 0,
                       act.has_value() ? typed(*act, "act") : 1, ids.has_value() ? ids->data_ptr<int>() : nullptr,
                       wts.has_value() ? f32w(wt, "wts") : nullptr, T, cur_stream()),
         "moe_route");
@@ -559,17 +562,81 @@ void latent_kv_write(const Tensor& q, int64_t H, int64_t dn, int64_t dr, const T
         "latent_kv_write");
 }
 
+// ---- stream whose mixer and feed-forward read the same x ----
+void parallel_boundary(const c10::optional<Tensor>& x_in, const Tensor& embed, const Tensor& tok, const c10::optional<Tensor>& o,
+                       const c10::optional<Tensor>& y, const c10::optional<Tensor>& slot_of, const c10::optional<Tensor>& w1,
+                       const c10::optional<Tensor>& w2, const c10::optional<Tensor>& mu, double eps, c10::optional<Tensor> x_out,
+                       c10::optional<Tensor> raw, c10::optional<Tensor> h1, c10::optional<Tensor> h2, const Tensor& cu, const Tensor& tok_entry,
+                       const Tensor& start, const Tensor& state_slot, const c10::optional<Tensor>& state, c10::optional<Tensor> carry,
+                       const c10::optional<Tensor>& commit, c10::optional<Tensor> commit_state) {
+  c10::cuda::CUDAGuard guard(embed.device());
+  const int T = static_cast<int>(tok.numel()), W = static_cast<int>(embed.size(1)), E = static_cast<int>(start.numel());
+  TORCH_CHECK(embed.dim() == 2 && embed.is_contiguous(), "parallel_boundary: embed [V, W]");
+  TORCH_CHECK(cu.numel() == E + 1 && tok_entry.numel() >= T && state_slot.numel() == E, "parallel_boundary: plan");
+  auto rows = [&](const c10::optional<Tensor>& t, const char* n, int64_t r) {          // float [r, W]
+    if (!t.has_value()) return static_cast<const float*>(nullptr);
+    TORCH_CHECK(t->dim() == 2 && t->is_contiguous() && t->size(1) == W && (r < 0 || t->size(0) == r), "parallel_boundary: ", n, " [", r, ", W]");
+    return f32(*t, n);
+  };
+  auto vec = [&](const c10::optional<Tensor>& t, const char* n) {
+    if (!t.has_value()) return static_cast<const float*>(nullptr);
+    TORCH_CHECK(t->numel() == W && t->is_contiguous(), "parallel_boundary: ", n, " [W]");
+    return f32(*t, n);
+  };
+  int h_f32 = -1;
+  auto operand = [&](c10::optional<Tensor>& t, const char* n) {                        // typed [T, W], all of one type
+    if (!t.has_value()) return static_cast<void*>(nullptr);
+    TORCH_CHECK(t->dim() == 2 && t->is_contiguous() && t->size(0) == T && t->size(1) == W, "parallel_boundary: ", n, " [T, W]");
+    const int f = typed(*t, n);
+    TORCH_CHECK(h_f32 < 0 || h_f32 == f, "parallel_boundary: raw, h1 and h2 have one type");
+    h_f32 = f;
+    return t->data_ptr();
+  };
+  void* rp = operand(raw, "raw");
+  void* p1 = operand(h1, "h1");
+  void* p2 = operand(h2, "h2");
+  TORCH_CHECK(y.has_value() == slot_of.has_value(), "parallel_boundary: y and slot_of go together");
+  int top = 0;
+  if (y.has_value()) {
+    TORCH_CHECK(T > 0 && slot_of->numel() % T == 0 && slot_of->numel() == y->size(0), "parallel_boundary: slot_of [T, top] names the rows of y");
+    top = static_cast<int>(slot_of->numel() / T);
+  }
+  const float* cs = rows(commit_state, "commit_state", -1);
+  const float* st = rows(state, "state", -1);
+  check(nrl_parallel_boundary(rows(x_in, "x_in", T), x_in.has_value() ? nullptr : embed.data_ptr(), typed(embed, "embed"), i32(tok, "tok"),
+                              rows(o, "o", T), rows(y, "y", -1), slot_of.has_value() ? i32(*slot_of, "slot_of") : nullptr, top, vec(w1, "w1"),
+                              vec(w2, "w2"), vec(mu, "mu"), static_cast<float>(eps), const_cast<float*>(rows(x_out, "x_out", T)), rp, p1, p2,
+                              h_f32 == 1 ? 1 : 0, i32(cu, "cu"), i32(tok_entry, "tok_entry"), i32(start, "start"),
+                              i32(state_slot, "state_slot"), st, const_cast<float*>(rows(carry, "carry", E)), rows(commit, "commit", E),
+                              const_cast<float*>(cs), T, W, cur_stream()),
+        "parallel_boundary");
+}
+
+void gate_cols(const Tensor& in, const Tensor& gate, double scale, Tensor out) {
+  c10::cuda::CUDAGuard guard(out.device());
+  TORCH_CHECK(in.dim() == 2 && out.dim() == 2 && gate.dim() == 2 && in.sizes() == out.sizes() && gate.sizes() == out.sizes(), "gate_cols: shapes");
+  check(nrl_gate_cols(f32(in, "in"), in.stride(0), f32(gate, "gate"), gate.stride(0), static_cast<float>(scale), out.data_ptr(), out.stride(0),
+                      typed(out, "out"), static_cast<int>(in.size(0)), static_cast<int>(in.size(1)), cur_stream()),
+        "gate_cols");
+}
+
 // ---- mixture of experts, grouped form ----
-std::vector<Tensor> moe_plan(const Tensor& ids, int64_t E, int64_t tile_rows, int64_t n_real) {
+std::vector<Tensor> moe_plan(const Tensor& ids, int64_t E, int64_t tile_rows, int64_t n_real, const c10::optional<Tensor>& wts,
+                             const c10::optional<Tensor>& row_weight) {
   c10::cuda::CUDAGuard guard(ids.device());
   TORCH_CHECK(ids.dim() == 2 && ids.scalar_type() == torch::kInt32 && ids.is_contiguous(), "moe_plan: ids int32 [T, top]");
   const int R = static_cast<int>(ids.numel()), top = static_cast<int>(ids.size(1));
+  TORCH_CHECK(wts.has_value() == row_weight.has_value(), "moe_plan: wts and row_weight go together");
+  if (wts.has_value())
+    TORCH_CHECK(wts->numel() == R && wts->is_contiguous() && row_weight->numel() == R && row_weight->is_contiguous(), "moe_plan: wts / row_weight [R]");
+  Tensor rw = row_weight.has_value() ? *row_weight : Tensor();
   const int64_t max_tiles = (R + tile_rows - 1) / tile_rows + E;
   auto opt = ids.options();
   Tensor slot_of = at::empty({R}, opt), row_token = at::empty({R}, opt), seg = at::empty({E + 1}, opt);
   Tensor tiles = at::zeros({max_tiles, 3}, opt), num_tiles = at::zeros({1}, opt);
-  check(nrl_moe_plan(i32(ids, "ids"), R, top, static_cast<int>(E), static_cast<int>(n_real < 0 ? E : n_real), static_cast<int>(tile_rows), slot_of.data_ptr<int>(),
-                     row_token.data_ptr<int>(), seg.data_ptr<int>(), tiles.data_ptr<int>(), num_tiles.data_ptr<int>(), cur_stream()),
+  check(nrl_moe_plan(i32(ids, "ids"), R, top, static_cast<int>(E), static_cast<int>(n_real < 0 ? E : n_real), static_cast<int>(tile_rows),
+                     wts.has_value() ? f32(*wts, "wts") : nullptr, slot_of.data_ptr<int>(), row_token.data_ptr<int>(),
+                     row_weight.has_value() ? f32w(rw, "row_weight") : nullptr, seg.data_ptr<int>(), tiles.data_ptr<int>(), num_tiles.data_ptr<int>(), cur_stream()),
         "moe_plan");
   return {slot_of, row_token, seg, tiles, num_tiles};
 }
@@ -584,11 +651,12 @@ void gather_rows(const Tensor& in, const Tensor& row_token, Tensor out) {
         "gather_rows");
 }
 
-void swiglu_rows(const Tensor& gu, Tensor act) {
+void swiglu_rows(const Tensor& gu, Tensor act, const c10::optional<Tensor>& row_scale) {
   c10::cuda::CUDAGuard guard(gu.device());
   TORCH_CHECK(gu.dim() == 2 && act.dim() == 2 && act.scalar_type() == torch::kBFloat16 && act.stride(1) == 1 && gu.size(0) == act.size(0) &&
                   gu.size(1) == 2 * act.size(1), "swiglu_rows: gu float [R, 2 ff], act bf16 [R, ff]");
-  check(nrl_swiglu_rows(f32(gu, "gu"), gu.stride(0), act.data_ptr(), act.stride(0), static_cast<int>(gu.size(0)),
+  if (row_scale.has_value()) TORCH_CHECK(row_scale->numel() == gu.size(0) && row_scale->is_contiguous(), "swiglu_rows: row_scale [R]");
+  check(nrl_swiglu_rows(f32(gu, "gu"), gu.stride(0), row_scale.has_value() ? f32(*row_scale, "row_scale") : nullptr, act.data_ptr(), act.stride(0), static_cast<int>(gu.size(0)),
                         static_cast<int>(act.size(1)), cur_stream()),
         "swiglu_rows");
 }
@@ -604,9 +672,9 @@ void moe_combine(const Tensor& y, const Tensor& slot_of, const Tensor& wts, Tens
 
 // Rows sorted by expert: a bf16 [R, K], b bf16 [E * N, K]; tiles / num_tiles from moe_plan (128-row tiles).
 //   out float [R, N] = a[r] . b[expert(r)]^T,  or
-//   act bf16 [R, N / 2] = silu(gate) * up with b's rows interleaved per 32 features ([32 gate rows | 32 up rows], N % 64 == 0).
+//   (row_scale float [R] then multiplies gate and up first)  act bf16 [R, N / 2] = silu(gate) * up with b's rows interleaved per 32 features ([32 gate rows | 32 up rows], N % 64 == 0).
 void gemm_tc_grouped(const Tensor& a, const Tensor& b, const c10::optional<Tensor>& out, const Tensor& tiles, const Tensor& num_tiles,
-                     int64_t block_n, const c10::optional<Tensor>& act) {
+                     int64_t block_n, const c10::optional<Tensor>& act, const c10::optional<Tensor>& row_scale) {
   c10::cuda::CUDAGuard guard(a.device());
   TORCH_CHECK(a.is_cuda() && b.is_cuda() && a.scalar_type() == torch::kBFloat16 && b.scalar_type() == torch::kBFloat16 && a.dim() == 2 &&
                   b.dim() == 2 && a.stride(1) == 1 && b.stride(1) == 1, "gemm_tc_grouped: bf16 2D operands with unit inner stride");
@@ -631,6 +699,10 @@ void gemm_tc_grouped(const Tensor& a, const Tensor& b, const c10::optional<Tenso
     p.out_bf16 = reinterpret_cast<__nv_bfloat16*>(act->data_ptr());
     p.out_stride = act->stride(0);
   }
+  if (row_scale.has_value()) {
+    TORCH_CHECK(act.has_value() && row_scale->numel() == R && row_scale->is_contiguous(), "gemm_tc_grouped: row_scale [R] goes with act");
+    p.row_scale = f32(*row_scale, "row_scale");
+  }
   if (R == 0) return;
   const int bn = block_n > 0 ? static_cast<int>(block_n) : (N <= 64 ? 64 : 128);
   const auto BF = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
@@ -652,13 +724,15 @@ void gemm_tc_grouped(const Tensor& a, const Tensor& b, const c10::optional<Tenso
 namespace nrl {
 void bind_hybrid(pybind11::module_& m) {
   m.def("moe_plan", &moe_plan, "sort (token, choice) pairs by expert: slot_of, row_token, seg, tiles, num_tiles (experts >= n_real get no tiles)",
-        pybind11::arg("ids"), pybind11::arg("E"), pybind11::arg("tile_rows"), pybind11::arg("n_real") = -1);
+        pybind11::arg("ids"), pybind11::arg("E"), pybind11::arg("tile_rows"), pybind11::arg("n_real") = -1, pybind11::arg("wts") = pybind11::none(),
+        pybind11::arg("row_weight") = pybind11::none());
   m.def("gather_rows", &gather_rows, "out[r] = in[row_token[r]] (bf16 rows)");
-  m.def("swiglu_rows", &swiglu_rows, "act = silu(gu[:, :ff]) * gu[:, ff:] (float in, bf16 out)");
+  m.def("swiglu_rows", &swiglu_rows, "act = silu(gu[:, :ff]) * gu[:, ff:] (float in, bf16 out)", pybind11::arg("gu"),
+        pybind11::arg("act"), pybind11::arg("row_scale") = pybind11::none());
   m.def("moe_combine", &moe_combine, "out[t] = sum_k wts[t, k] y[slot_of[t, k]]");
   m.def("gemm_tc_grouped", &gemm_tc_grouped, "grouped tcgen05 GEMM over rows sorted by expert: float32 out, or fused SwiGLU bf16 out",
         pybind11::arg("a"), pybind11::arg("b"), pybind11::arg("out"), pybind11::arg("tiles"), pybind11::arg("num_tiles"),
-        pybind11::arg("block_n") = 0, pybind11::arg("act") = pybind11::none());
+        pybind11::arg("block_n") = 0, pybind11::arg("act") = pybind11::none(), pybind11::arg("row_scale") = pybind11::none());
   m.def("embed_norm", &embed_norm, "x = rmsnorm(embed[tok]) * w (float), h = x (typed)");
   m.def("post_norm_residual", &post_norm_residual, "x += rmsnorm(o + self_w x) * w_post; h = w_pre ? rmsnorm(x) * w_pre : x");
   m.def("side_gate", &side_gate, "out = gelu_tanh(u) * table[tok, col0:col0 + C], zero padded");
@@ -694,6 +768,11 @@ void bind_hybrid(pybind11::module_& m) {
   m.def("kv_write_blend", &kv_write_blend, "keys and (optionally blended) values of a step's tokens into their pages");
   m.def("embed_hashed", &embed_hashed, "x0 = embed[tok] * scale + pair[hash(previous token, token)] (float), previous tokens carried per slot");
   m.def("group_norm_residual", &group_norm_residual, "x += groupnorm(o * sigmoid(gate)) * w_post; h = groupnorm(x) * w_pre");
-  m.def("moe_route", &moe_route, "top-k routing with softmax over the chosen logits; dense-form expert activations");
+  m.def("moe_route", &moe_route, "top-k routing with softmax over the chosen logits or their sigmoids; dense-form expert activations",
+        pybind11::arg("router"), pybind11::arg("router_bias"), pybind11::arg("top"), pybind11::arg("gu"), pybind11::arg("ff"),
+        pybind11::arg("act"), pybind11::arg("ids"), pybind11::arg("wts"), pybind11::arg("sigmoid") = false,
+        pybind11::arg("weight_input") = false);
+  m.def("parallel_boundary", &parallel_boundary, "x += results; two RMS norms of x, the first with a token shift carried per slot");
+  m.def("gate_cols", &gate_cols, "out = scale * in * sigmoid(gate)");
 }
 }  // namespace nrl

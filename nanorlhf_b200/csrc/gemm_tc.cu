@@ -448,14 +448,15 @@ NRL_DEVICE void gemm_tc_body(const CUtensorMap& tmA, const CUtensorMap& tmB, con
           // in every 64-column chunk), so a chunk yields 32 activations of this row: 64 contiguous bytes, plain masked stores
           const int f0 = c.n_blk * (BN / 2) + ch * 32;
           if (row_ok && f0 < p.N / 2) {
+            const float rw = p.row_scale != nullptr ? p.row_scale[row] : 1.f;      // a weight on the expert's input: gate and up scale with it
             __nv_bfloat16* orow = p.out_bf16 + static_cast<long>(row) * p.out_stride + f0;
 #pragma unroll
             for (int j = 0; j < 32; j += 8) {
               uint32_t pk[4];
 #pragma unroll
               for (int e = 0; e < 4; ++e) {
-                const float g0 = __uint_as_float(v[0][j + 2 * e]), g1 = __uint_as_float(v[0][j + 2 * e + 1]);
-                const float u0 = __uint_as_float(v[1][j + 2 * e]), u1 = __uint_as_float(v[1][j + 2 * e + 1]);
+                const float g0 = rw * __uint_as_float(v[0][j + 2 * e]), g1 = rw * __uint_as_float(v[0][j + 2 * e + 1]);
+                const float u0 = rw * __uint_as_float(v[1][j + 2 * e]), u1 = rw * __uint_as_float(v[1][j + 2 * e + 1]);
                 pk[e] = pack_bf16x2(g0 / (1.f + __expf(-g0)) * u0, g1 / (1.f + __expf(-g1)) * u1);
               }
               *reinterpret_cast<uint4*>(orow + j) = make_uint4(pk[0], pk[1], pk[2], pk[3]);

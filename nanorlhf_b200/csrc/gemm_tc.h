@@ -16,7 +16,7 @@ enum TcEpilogue : int {
 struct TcParams {
   int M, N, K;                  // D is [M, N]; K = contraction length of the first operand pair
   int K2;                       // contraction length of the second operand pair (0 = none)
-  const float* row_scale;       // FP8 kernels: [M] per-token dequantisation scale of A
+  const float* row_scale;       // FP8 kernels: [M] per-token dequantisation scale of A (GROUPED: see below)
   const float* col_scale;       // FP8 kernels: [N] per-output-channel dequantisation scale of B
   int batch;                    // BATCH kernels: number of independent [M,K] x [N,K]^T problems behind 3D tensor maps (else 1)
   float alpha;                  // multiplies the accumulator
@@ -54,7 +54,7 @@ extern "C" cudaError_t nrl_gemm_tc_batched(const CUtensorMap* maps, const nrl::t
 // grouped K-major x K-major GEMM (cta_group 1); maps = {A [rows, K] box {128, 64}, B [experts * N, K] box {bn, 64}};
 // p->N = columns per expert; max_tiles bounds the table's length (grid size).  Output: out_f32 [rows, N], or, when out_bf16 is
 // set, the SwiGLU of the columns: B rows interleaved per 32 features ([32 gate | 32 up], N % 64 == 0), out_bf16 [rows, N / 2]
-// (row stride out_stride, a multiple of 8) = silu(gate) * up.
+// (row stride out_stride, a multiple of 8) = silu(gate) * up; row_scale [rows] (or null) then multiplies gate and up first.
 extern "C" cudaError_t nrl_gemm_tc_grouped(const CUtensorMap* maps, const nrl::tc::TcParams* p, int bn, int max_tiles, int num_sms,
                                            cudaStream_t stream);
 extern "C" cudaError_t nrl_gemm_tc(const CUtensorMap* maps, const nrl::tc::TcParams* p, int cg, int bn, int a_mn, int b_mn,

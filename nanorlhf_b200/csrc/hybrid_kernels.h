@@ -55,24 +55,26 @@ cudaError_t nrl_group_norm_residual(float* x, const float* o, const float* gate,
                                     const float* w_pre, int groups, float eps, void* h, int h_f32, int T, int W, cudaStream_t s);
 
 // Mixture-of-experts routing.  router float [T, E] (row stride sr) + router_bias [E]; the `top` largest logits (ties: lowest
-// index) are chosen, weights = softmax over the chosen logits.  ids int [T, top], wts float [T, top] (either may be null).
+// index) are chosen, weights = softmax over the chosen logits, or (sigmoid) each chosen logit's own sigmoid.  ids int [T, top], wts float [T, top] (either may be null).
 // Dense form (act != nullptr): gu float (row stride sgu) holds per expert ff gate columns then ff up columns;
-//   act[t, e*ff + c] (typed, row stride sa) = weight_e * silu(gate) * up, 0 for experts that were not chosen.
-cudaError_t nrl_moe_route(const float* router, long sr, const float* router_bias, int E, int top, const float* gu, long sgu, int ff,
-                          void* act, long sa, int act_f32, int* ids, float* wts, int T, cudaStream_t s);
+//   act[t, e*ff + c] (typed, row stride sa) = weight_e * silu(gate) * up, 0 for experts that were not chosen; weight_input:
+//   silu(weight_e * gate) * (weight_e * up), the weight on the expert's input.
+cudaError_t nrl_moe_route(const float* router, long sr, const float* router_bias, int E, int top, int sigmoid, int weight_input,
+                          const float* gu, long sgu, int ff, void* act, long sa, int act_f32, int* ids, float* wts, int T, cudaStream_t s);
 
 // Grouped (sorted by expert) form of a mixture of experts, moe.cu.  ids int [R = T * top] from nrl_moe_route.
 //   nrl_moe_plan: slot_of[R] = row of every (token, choice) pair in expert order, row_token[R] = token of every row,
 //     seg[E + 1] = first row of every expert, tiles [*, 3] = (expert, first row, end row of the expert) per `tile_rows` rows of
 //     an expert (at most ceil(R / tile_rows) + E of them), num_tiles[1]: the table of the grouped GEMM (gemm_tc.h).
 //   nrl_gather_rows16: out[r] = in[row_token[r]] for rows of W 16-bit elements.
-//   nrl_swiglu_rows: act[r, c] (bf16) = silu(gu[r, c]) * gu[r, ff + c].
+//   nrl_swiglu_rows: act[r, c] (bf16) = silu(w gu[r, c]) * (w gu[r, ff + c]), w = row_scale[r] (null: 1).
 //   nrl_moe_combine: out[t] (float) = sum_k wts[t, k] * y[slot_of[t * top + k]] in the order of k.
 // n_real <= E: experts n_real .. E-1 get rows but no tiles (identity experts); nrl_moe_combine skips pairs of weight 0.
-cudaError_t nrl_moe_plan(const int* ids, int R, int top, int E, int n_real, int tile_rows, int* slot_of, int* row_token, int* seg, int* tiles,
-                         int* num_tiles, cudaStream_t s);
+// wts [R] with row_weight [R] (both or neither): the pairs' weights in expert order.
+cudaError_t nrl_moe_plan(const int* ids, int R, int top, int E, int n_real, int tile_rows, const float* wts, int* slot_of, int* row_token,
+                         float* row_weight, int* seg, int* tiles, int* num_tiles, cudaStream_t s);
 cudaError_t nrl_gather_rows16(const void* in, long in_stride, const int* row_token, void* out, int R, int W, cudaStream_t s);
-cudaError_t nrl_swiglu_rows(const float* gu, long sg, void* act, long sa, int R, int ff, cudaStream_t s);
+cudaError_t nrl_swiglu_rows(const float* gu, long sg, const float* row_scale, void* act, long sa, int R, int ff, cudaStream_t s);
 cudaError_t nrl_moe_combine(const float* y, long sy, const int* slot_of, const float* wts, int top, float* out, long so, int T, int W,
                             cudaStream_t s);
 
@@ -113,7 +115,7 @@ cudaError_t nrl_act_cols(const float* in, long si, void* out, long so, int out_f
 
 // Part-wise gated RMS norm:  y [T, n] float (row stride sy), gate float (row stride sg).  Parts of `part` columns.
 //   gate_first: v = y * act(gate); v /= rms_part(v); v *= w        else: v = y / rms_part(y) * w * act(gate)
-//   w index = shared_w ? (c % part) : c.   gate_act: 0 silu, 1 sigmoid.   out typed = scale * v
+//   w index = shared_w ? (c % part) : c.   gate_act: 0 silu, 1 sigmoid.   out typed = scale * v.   gate null: no gate
 cudaError_t nrl_gated_part_rmsnorm(const float* y, long sy, const float* gate, long sg, const float* w, int shared_w, int part,
                                    int gate_act, int gate_first, float eps, float scale, void* out, long so, int out_f32,
                                    int T, int n, cudaStream_t s);
@@ -218,6 +220,22 @@ cudaError_t nrl_window_attention_mma(const float* q, long sq, const void* k_cach
                                      int max_blocks, const int* tok_entry, const int* pos, int window, float scale, float out_scale,
                                      void* out, long so, int T, int Hq, int Hkv, int D, int Dv, int page, int single_token,
                                      const NrlAttnMods* mods, cudaStream_t s);
+// Boundary of a stream whose mixer and feed-forward read the same x side by side, each behind its own RMS norm (weights per column).
+//   x = (x_in [T, W], or embed[tok] when x_in is null) + o [T, W] + sum_k y[slot_of[t * top + k]]      (o, y may be null)
+//   x_out (float, not x_in) = x;  raw (typed) = x;  h1 (typed) = x / rms(x) * w1;  h2 (typed) = x / rms(x) * w2      (any may be null)
+//   mu [W] (or null), token shift: h1 <- h1 + (h1 of the sequence's previous token - h1) * mu;  the previous token's h1 of an entry's
+//   first token is its slot's row of state [slots, W] (zeros at position 0);  the last token's h1 goes to carry [entries, W]
+//   commit [entries, W] -> commit_state [slots, W]: hands an EARLIER boundary's carry to its state (one launch never writes the
+//   state it reads)
+cudaError_t nrl_parallel_boundary(const float* x_in, const void* embed, int w_f32, const int* tok, const float* o, const float* y,
+                                  const int* slot_of, int top, const float* w1, const float* w2, const float* mu, float eps, float* x_out,
+                                  void* raw, void* h1, void* h2, int h_f32, const int* cu, const int* tok_entry, const int* start,
+                                  const int* state_slot, const float* state, float* carry, const float* commit, float* commit_state, int T,
+                                  int W, cudaStream_t s);
+// out[t, c] (typed, row stride so) = scale * in[t, c] * sigmoid(gate[t, c])  (floats, row strides si / sg)
+cudaError_t nrl_gate_cols(const float* in, long si, const float* gate, long sg, float scale, void* out, long so, int out_f32, int T, int C,
+                          cudaStream_t s);
+
 // Several residual streams mixed by learned weights (hyper-connections), layer norms with weight and bias.  xs float [T, S, W].
 //   nrl_embed_streams:   xs[t, s] = embed[tok[t]] * scale for every stream s
 //   nrl_hyper_boundary:  if (o)  y = o + o_bias + self_w[t] * h[t]  (o float [T, W]; o_bias [W], self_w [T] or null; h still holds

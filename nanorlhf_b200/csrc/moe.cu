@@ -12,9 +12,10 @@ namespace {
 
 // One block.  ids [R] (R = tokens * top): expert of every pair.  Outputs: slot_of[R] (row of the pair in expert order),
 // row_token[R] (token of every row), seg[E + 1] (first row of every expert), tiles [*, 3] = (expert, first row, end row of the
-// expert) for every `tile_rows` rows of every expert that has rows, num_tiles[1].
-__global__ void moe_plan_kernel(const int* __restrict__ ids, int R, int top, int E, int n_real, int tile_rows, int* __restrict__ slot_of,
-                                int* __restrict__ row_token, int* __restrict__ seg, int* __restrict__ tiles, int* __restrict__ num_tiles) {
+// expert) for every `tile_rows` rows of every expert that has rows, num_tiles[1].  row_weight[R] (if not null): wts [R] in expert order.
+__global__ void moe_plan_kernel(const int* __restrict__ ids, int R, int top, int E, int n_real, int tile_rows,
+                                const float* __restrict__ wts, int* __restrict__ slot_of, int* __restrict__ row_token,
+                                float* __restrict__ row_weight, int* __restrict__ seg, int* __restrict__ tiles, int* __restrict__ num_tiles) {
   extern __shared__ int sh[];
   int* cnt = sh;             // [E]
   int* start = sh + E;       // [E + 1]
@@ -48,6 +49,7 @@ __global__ void moe_plan_kernel(const int* __restrict__ ids, int R, int top, int
     const int s = atomicAdd(&cnt[ids[i]], 1);     // the order of an expert's rows is arbitrary: rows are independent
     slot_of[i] = s;
     row_token[s] = i / top;
+    if (row_weight != nullptr) row_weight[s] = wts[i];
   }
 }
 
@@ -62,14 +64,19 @@ __global__ void gather_rows_kernel(const uint4* __restrict__ in, long in_stride1
   }
 }
 
-// act[r, c] (bf16) = silu(gu[r, c]) * gu[r, ff + c];  four columns per thread
-__global__ void swiglu_rows_kernel(const float* __restrict__ gu, long sg, __nv_bfloat16* __restrict__ act, long sa, int R, int ff4) {
+// act[r, c] (bf16) = silu(w gu[r, c]) * (w gu[r, ff + c]) with w = row_scale[r] (null: 1);  four columns per thread
+__global__ void swiglu_rows_kernel(const float* __restrict__ gu, long sg, const float* __restrict__ row_scale, __nv_bfloat16* __restrict__ act, long sa, int R, int ff4) {
   const long n = static_cast<long>(R) * ff4;
   for (long idx = blockIdx.x * static_cast<long>(blockDim.x) + threadIdx.x; idx < n; idx += static_cast<long>(gridDim.x) * blockDim.x) {
     const long r = idx / ff4;
     const int c = static_cast<int>(idx - r * ff4) * 4;
-    const float4 g = *reinterpret_cast<const float4*>(gu + r * sg + c);
-    const float4 u = *reinterpret_cast<const float4*>(gu + r * sg + ff4 * 4 + c);
+    float4 g = *reinterpret_cast<const float4*>(gu + r * sg + c);
+    float4 u = *reinterpret_cast<const float4*>(gu + r * sg + ff4 * 4 + c);
+    if (row_scale != nullptr) {
+      const float w = row_scale[r];
+      g.x *= w; g.y *= w; g.z *= w; g.w *= w;
+      u.x *= w; u.y *= w; u.z *= w; u.w *= w;
+    }
     const float a0 = g.x / (1.f + expf(-g.x)) * u.x, a1 = g.y / (1.f + expf(-g.y)) * u.y;
     const float a2 = g.z / (1.f + expf(-g.z)) * u.z, a3 = g.w / (1.f + expf(-g.w)) * u.w;
     const __nv_bfloat162 lo = __floats2bfloat162_rn(a0, a1), hi = __floats2bfloat162_rn(a2, a3);
@@ -107,11 +114,13 @@ inline int grid_for(long n, int threads) {
 
 extern "C" {
 
-cudaError_t nrl_moe_plan(const int* ids, int R, int top, int E, int n_real, int tile_rows, int* slot_of, int* row_token, int* seg, int* tiles,
-                         int* num_tiles, cudaStream_t s) {
+cudaError_t nrl_moe_plan(const int* ids, int R, int top, int E, int n_real, int tile_rows, const float* wts, int* slot_of, int* row_token,
+                         float* row_weight, int* seg, int* tiles, int* num_tiles, cudaStream_t s) {
   if (R <= 0) return cudaSuccess;
-  if (E < 1 || E > 8192 || top < 1 || tile_rows < 1 || n_real < 0 || n_real > E) return cudaErrorInvalidValue;
-  moe_plan_kernel<<<1, 1024, sizeof(int) * (2 * E + 1), s>>>(ids, R, top, E, n_real, tile_rows, slot_of, row_token, seg, tiles, num_tiles);
+  if (E < 1 || E > 8192 || top < 1 || tile_rows < 1 || n_real < 0 || n_real > E || (row_weight != nullptr && wts == nullptr))
+    return cudaErrorInvalidValue;
+  moe_plan_kernel<<<1, 1024, sizeof(int) * (2 * E + 1), s>>>(ids, R, top, E, n_real, tile_rows, wts, slot_of, row_token, row_weight, seg, tiles,
+                                                          num_tiles);
   return cudaGetLastError();
 }
 
@@ -124,12 +133,12 @@ cudaError_t nrl_gather_rows16(const void* in, long in_stride, const int* row_tok
   return cudaGetLastError();
 }
 
-cudaError_t nrl_swiglu_rows(const float* gu, long sg, void* act, long sa, int R, int ff, cudaStream_t s) {
+cudaError_t nrl_swiglu_rows(const float* gu, long sg, const float* row_scale, void* act, long sa, int R, int ff, cudaStream_t s) {
   if (R <= 0) return cudaSuccess;
   if (ff % 4 != 0 || sg % 4 != 0 || sa % 4 != 0 || reinterpret_cast<uintptr_t>(gu) % 16 != 0 || reinterpret_cast<uintptr_t>(act) % 8 != 0)
     return cudaErrorInvalidValue;
   const long n = static_cast<long>(R) * (ff / 4);
-  swiglu_rows_kernel<<<grid_for(n, 256), 256, 0, s>>>(gu, sg, static_cast<__nv_bfloat16*>(act), sa, R, ff / 4);
+  swiglu_rows_kernel<<<grid_for(n, 256), 256, 0, s>>>(gu, sg, row_scale, static_cast<__nv_bfloat16*>(act), sa, R, ff / 4);
   return cudaGetLastError();
 }
 

@@ -272,13 +272,15 @@ __global__ void group_norm_residual_vec_kernel(float* __restrict__ x, const floa
 }
 
 // Mixture-of-experts routing and (dense form) expert activations, one block per token.
-//   z = router[t, :E] + router_bias;  the `top` largest (ties: lowest index) get softmax(z over the chosen) as weights
+//   z = router[t, :E] + router_bias;  the `top` largest (ties: lowest index) get softmax(z over the chosen) as weights, or
+//   (sigmoid) each its own sigmoid(z)
 //   ids [T, top] int, wts [T, top] float (if not null)
-//   act != nullptr:  act[t, e*ff + c] = weight_e * silu(gu[t, e*2ff + c]) * gu[t, e*2ff + ff + c], 0 for experts not chosen
+//   act != nullptr:  act[t, e*ff + c] = weight_e * silu(gu[t, e*2ff + c]) * gu[t, e*2ff + ff + c], 0 for experts not chosen;
+//   weight_input: the weight multiplies the expert's input, i.e. (the projections being linear) both columns before the activation
 template <typename OT>
 __global__ void moe_route_kernel(const float* __restrict__ router, long sr, const float* __restrict__ router_bias, int E, int top,
-                                 const float* __restrict__ gu, long sgu, int ff, OT* __restrict__ act, long sa, int* __restrict__ ids,
-                                 float* __restrict__ wts) {
+                                 int sigmoid, int weight_input, const float* __restrict__ gu, long sgu, int ff, OT* __restrict__ act, long sa,
+                                 int* __restrict__ ids, float* __restrict__ wts) {
   extern __shared__ float smf[];
   float* z = smf;                 // [E]
   float* wsel = z + E;            // [E]: weight, 0 = not chosen
@@ -305,7 +307,7 @@ __global__ void moe_route_kernel(const float* __restrict__ router, long sr, cons
         if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
       }
       if (k == 0) zmax = best;
-      const float p = expf(best - zmax);
+      const float p = sigmoid ? sigmoidf_(best) : expf(best - zmax);
       denom += p;
       __syncwarp();
       if (lane == 0) {
@@ -315,7 +317,8 @@ __global__ void moe_route_kernel(const float* __restrict__ router, long sr, cons
       }
       __syncwarp();
     }
-    for (int e = lane; e < E; e += 32) wsel[e] = wsel[e] / denom;
+    if (!sigmoid)
+      for (int e = lane; e < E; e += 32) wsel[e] = wsel[e] / denom;
     __syncwarp();
     if (wts != nullptr)
       for (int k = lane; k < top; k += 32) wts[t * top + k] = wsel[ids[t * top + k]];
@@ -329,7 +332,7 @@ __global__ void moe_route_kernel(const float* __restrict__ router, long sr, cons
     float v = 0.f;
     if (w != 0.f) {
       const float gt = gu[t * sgu + static_cast<long>(e) * 2 * ff + c], up = gu[t * sgu + static_cast<long>(e) * 2 * ff + ff + c];
-      v = w * (gt * sigmoidf_(gt) * up);
+      v = weight_input ? w * gt * sigmoidf_(w * gt) * (w * up) : w * (gt * sigmoidf_(gt) * up);
     }
     st(act, t * sa + idx, v);
   }
@@ -631,7 +634,7 @@ __global__ void gated_part_rmsnorm_kernel(const float* __restrict__ y, long sy, 
   const long t = wid / nparts;
   const int p = static_cast<int>(wid - t * nparts);
   const float* yr = y + t * sy + static_cast<long>(p) * part;
-  const float* gr = gate + t * sg + static_cast<long>(p) * part;
+  const float* gr = gate != nullptr ? gate + t * sg + static_cast<long>(p) * part : nullptr;
   float ss = 0.f;
   for (int c = lane * V; c < part; c += 32 * V) {
     float v[V], gv[V];
@@ -648,11 +651,11 @@ __global__ void gated_part_rmsnorm_kernel(const float* __restrict__ y, long sy, 
   for (int c = lane * V; c < part; c += 32 * V) {
     float v[V], gv[V], wv[V];
     ldv<V>(yr + c, v);
-    ldv<V>(gr + c, gv);
+    if (gate != nullptr) ldv<V>(gr + c, gv);
     ldv<V>(w + (shared_w ? c : p * part + c), wv);
 #pragma unroll
     for (int i = 0; i < V; ++i) {
-      const float gg = gate_fn(gv[i], gate_act);
+      const float gg = gate != nullptr ? gate_fn(gv[i], gate_act) : 1.f;
       v[i] = scale * (gate_first ? (v[i] * gg) * r * wv[i] : v[i] * r * wv[i] * gg);
     }
     stv<V>(out + t * so + static_cast<long>(p) * part + c, v);
@@ -669,7 +672,7 @@ __global__ void gated_part_rmsnorm_block_kernel(const float* __restrict__ y, lon
   const int p = static_cast<int>(blockIdx.x - t * nparts);
   const int lane = threadIdx.x & 31, wi = threadIdx.x >> 5, nw = blockDim.x >> 5;
   const float* yr = y + t * sy + static_cast<long>(p) * part;
-  const float* gr = gate + t * sg + static_cast<long>(p) * part;
+  const float* gr = gate != nullptr ? gate + t * sg + static_cast<long>(p) * part : nullptr;
   float ss = 0.f;
   for (int c = threadIdx.x * V; c < part; c += blockDim.x * V) {
     float v[V], gv[V];
@@ -690,11 +693,11 @@ __global__ void gated_part_rmsnorm_block_kernel(const float* __restrict__ y, lon
   for (int c = threadIdx.x * V; c < part; c += blockDim.x * V) {
     float v[V], gv[V], wv[V];
     ldv<V>(yr + c, v);
-    ldv<V>(gr + c, gv);
+    if (gate != nullptr) ldv<V>(gr + c, gv);
     ldv<V>(w + (shared_w ? c : p * part + c), wv);
 #pragma unroll
     for (int i = 0; i < V; ++i) {
-      const float gg = gate_fn(gv[i], gate_act);
+      const float gg = gate != nullptr ? gate_fn(gv[i], gate_act) : 1.f;
       v[i] = scale * (gate_first ? (v[i] * gg) * r * wv[i] : v[i] * r * wv[i] * gg);
     }
     stv<V>(out + t * so + static_cast<long>(p) * part + c, v);
@@ -736,6 +739,156 @@ __global__ void embed_streams_kernel(const WT* __restrict__ embed, const int* __
   for (int c = threadIdx.x; c < W; c += blockDim.x) {
     const float v = ld(row, c) * scale;
     for (int s = 0; s < S; ++s) xs[(t * S + s) * W + c] = v;
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// Stream whose mixer and feed-forward read the same x, each behind its own RMS norm, with an optional token shift of the mixer's
+// input: h1 <- h1 + (previous token's h1 - h1) * mu.
+// ---------------------------------------------------------------------------------------------------------------------
+// A block owns `rows` consecutive tokens; a thread owns fixed columns, so the row buffers in shared memory are thread-private.
+//   x = (x_in or embed[tok]) + o[t] + sum_k y[slot_of[t * top + k]]
+//   x_out = x (float);  raw = x (typed);  h1 = shift(x / rms(x) * w1) (typed);  h2 = x / rms(x) * w2 (typed);  any may be null
+// The previous token's h1 comes from the row above: the block's own, recomputed for the first row of a block, or, for the first
+// token of an entry, the sequence's slot of `state` (zeros at position 0).  The h1 of an entry's last token goes to `carry` [entries, W] and
+// reaches the slot with the NEXT boundary of the step (its `commit` / `commit_state`): the blocks of one launch read the old state.
+struct ParallelBoundary {
+  const float* x_in;
+  const void* embed;
+  const int* tok;
+  const float* o;
+  const float* y;
+  const int* slot_of;
+  int top;
+  const float* w1;
+  const float* w2;
+  const float* mu;
+  float eps;
+  float* x_out;
+  void* raw;
+  void* h1;
+  void* h2;
+  const int* cu;
+  const int* tok_entry;
+  const int* start;
+  const int* state_slot;
+  const float* state;
+  float* carry;
+  const float* commit;
+  float* commit_state;
+  int T, W, rows;
+};
+
+template <typename WT, typename HT, int V>
+__global__ void __launch_bounds__(256) parallel_boundary_kernel(const ParallelBoundary p) {
+  extern __shared__ __align__(16) float rowbuf[];         // [2][W]: the row's x, the previous row's h1
+  __shared__ float red[32];
+  const int W = p.W;
+  float* cur = rowbuf;
+  float* prev = rowbuf + W;
+  const int t0 = blockIdx.x * p.rows, t1 = min(p.T, t0 + p.rows);
+  const bool shift = p.mu != nullptr && p.h1 != nullptr;
+  const bool norms = p.h1 != nullptr || p.h2 != nullptr;
+  const int step = blockDim.x * V;
+  bool above = false;                                      // the first row's predecessor is in this step: its h1 is formed again
+  if (shift) above = t0 > p.cu[p.tok_entry[t0]];
+  for (int t = above ? t0 - 1 : t0; t < t1; ++t) {
+    const bool own = t >= t0;
+    const long row = static_cast<long>(t) * W;
+    float ss = 0.f;
+    for (int c = threadIdx.x * V; c < W; c += step) {
+      float v[V], a[V];
+      if (p.x_in != nullptr) {
+        ldv<V>(p.x_in + row + c, v);
+      } else {
+        const WT* er = static_cast<const WT*>(p.embed) + static_cast<long>(p.tok[t]) * W + c;
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = ld(er, e);
+      }
+      if (p.o != nullptr) {
+        ldv<V>(p.o + row + c, a);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] += a[e];
+      }
+      if (p.y != nullptr) {
+        for (int k = 0; k < p.top; ++k) {
+          ldv<V>(p.y + static_cast<long>(p.slot_of[static_cast<long>(t) * p.top + k]) * W + c, a);
+#pragma unroll
+          for (int e = 0; e < V; ++e) v[e] += a[e];
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss += v[e] * v[e];
+      stv<V>(cur + c, v);
+      if (own && p.x_out != nullptr) stv<V>(p.x_out + row + c, v);
+      if (own && p.raw != nullptr) stv<V>(static_cast<HT*>(p.raw) + row + c, v);
+    }
+    const int e_id = p.tok_entry[t];
+    const bool last = own && t + 1 == p.cu[e_id + 1];
+    const long crow = static_cast<long>(e_id) * W;
+    if (last && p.commit != nullptr) {
+      const long srow = static_cast<long>(p.state_slot[e_id]) * W;
+      for (int c = threadIdx.x * V; c < W; c += step) {
+        float v[V];
+        ldv<V>(p.commit + crow + c, v);
+        stv<V>(p.commit_state + srow + c, v);
+      }
+    }
+    if (!norms) continue;
+    ss = block_sum(ss, red);
+    const float r = 1.f / sqrtf(ss / static_cast<float>(W) + p.eps);
+    const bool first = t == p.cu[e_id];
+    const bool fresh = first && p.start[e_id] == 0;
+    const long srow = shift && first ? static_cast<long>(p.state_slot[e_id]) * W : 0;
+    for (int c = threadIdx.x * V; c < W; c += step) {
+      float v[V], w[V], h[V];
+      ldv<V>(cur + c, v);
+      if (p.h1 != nullptr) {
+        ldv<V>(p.w1 + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[e] = v[e] * r * w[e];
+        if (shift) {
+          float q[V], mu[V], out[V];
+          if (fresh) {
+#pragma unroll
+            for (int e = 0; e < V; ++e) q[e] = 0.f;
+          } else {
+            ldv<V>(first ? p.state + srow + c : prev + c, q);
+          }
+          ldv<V>(p.mu + c, mu);
+#pragma unroll
+          for (int e = 0; e < V; ++e) out[e] = h[e] + (q[e] - h[e]) * mu[e];
+          stv<V>(prev + c, h);
+          if (own) stv<V>(static_cast<HT*>(p.h1) + row + c, out);
+          if (last) stv<V>(p.carry + crow + c, h);
+        } else {
+          stv<V>(static_cast<HT*>(p.h1) + row + c, h);
+        }
+      }
+      if (own && p.h2 != nullptr) {
+        ldv<V>(p.w2 + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[e] = v[e] * r * w[e];
+        stv<V>(static_cast<HT*>(p.h2) + row + c, h);
+      }
+    }
+  }
+}
+
+// out[t, c] (typed, row stride so) = scale * in[t, c] * sigmoid(gate[t, c]);  V columns per thread
+template <typename OT, int V>
+__global__ void gate_cols_kernel(const float* __restrict__ in, long si, const float* __restrict__ gate, long sg, float scale,
+                                 OT* __restrict__ out, long so, long T, int CV) {
+  const long n = T * CV;
+  for (long idx = blockIdx.x * static_cast<long>(blockDim.x) + threadIdx.x; idx < n; idx += static_cast<long>(gridDim.x) * blockDim.x) {
+    const long t = idx / CV;
+    const int c = static_cast<int>(idx - t * CV) * V;
+    float v[V], g[V];
+    ldv<V>(in + t * si + c, v);
+    ldv<V>(gate + t * sg + c, g);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = scale * v[e] * sigmoidf_(g[e]);
+    stv<V>(out + t * so + c, v);
   }
 }
 
@@ -914,17 +1067,18 @@ cudaError_t nrl_group_norm_residual(float* x, const float* o, const float* gate,
   return cudaGetLastError();
 }
 
-cudaError_t nrl_moe_route(const float* router, long sr, const float* router_bias, int E, int top, const float* gu, long sgu, int ff,
-                          void* act, long sa, int act_f32, int* ids, float* wts, int T, cudaStream_t s) {
+cudaError_t nrl_moe_route(const float* router, long sr, const float* router_bias, int E, int top, int sigmoid, int weight_input,
+                          const float* gu, long sgu, int ff, void* act, long sa, int act_f32, int* ids, float* wts, int T, cudaStream_t s) {
   if (T <= 0) return cudaSuccess;
   if (E < 1 || top < 1 || top > E || E > 4096 || (wts != nullptr && ids == nullptr)) return cudaErrorInvalidValue;
   const size_t smem = sizeof(float) * 2 * E;
   const int th = act == nullptr ? 32 : 256;
   if (act_f32)
-    moe_route_kernel<float><<<T, th, smem, s>>>(router, sr, router_bias, E, top, gu, sgu, ff, static_cast<float*>(act), sa, ids, wts);
+    moe_route_kernel<float><<<T, th, smem, s>>>(router, sr, router_bias, E, top, sigmoid, weight_input, gu, sgu, ff, static_cast<float*>(act),
+                                             sa, ids, wts);
   else
-    moe_route_kernel<__nv_bfloat16><<<T, th, smem, s>>>(router, sr, router_bias, E, top, gu, sgu, ff, static_cast<__nv_bfloat16*>(act),
-                                                        sa, ids, wts);
+    moe_route_kernel<__nv_bfloat16><<<T, th, smem, s>>>(router, sr, router_bias, E, top, sigmoid, weight_input, gu, sgu, ff,
+                                                     static_cast<__nv_bfloat16*>(act), sa, ids, wts);
   return cudaGetLastError();
 }
 
@@ -1056,10 +1210,10 @@ cudaError_t nrl_gated_part_rmsnorm(const float* y, long sy, const float* gate, l
                                    int gate_act, int gate_first, float eps, float scale, void* out, long so, int out_f32, int T,
                                    int n, cudaStream_t s) {
   if (T <= 0 || n <= 0) return cudaSuccess;
-  if (part <= 0 || n % part != 0) return cudaErrorInvalidValue;
+  if (part <= 0 || n % part != 0 || (gate == nullptr && gate_first)) return cudaErrorInvalidValue;
   const int nparts = n / part;
-  const bool vec = part % 4 == 0 && sy % 4 == 0 && sg % 4 == 0 && so % 4 == 0 && aligned(y, 16) && aligned(gate, 16) && aligned(w, 16) &&
-                   aligned(out, out_f32 ? 16 : 8);
+  const bool vec = part % 4 == 0 && sy % 4 == 0 && so % 4 == 0 && (gate == nullptr || (sg % 4 == 0 && aligned(gate, 16))) && aligned(y, 16) &&
+                   aligned(w, 16) && aligned(out, out_f32 ? 16 : 8);
 #define NRL_GN(OT_, V_)                                                                                                            \
   return launch_gated_norm<OT_, V_>(y, sy, gate, sg, w, shared_w, part, gate_act, gate_first, eps, scale, static_cast<OT_*>(out), so, T, \
                                     nparts, s)
@@ -1070,6 +1224,71 @@ cudaError_t nrl_gated_part_rmsnorm(const float* y, long sy, const float* gate, l
   if (vec) NRL_GN(__nv_bfloat16, 4);
   NRL_GN(__nv_bfloat16, 1);
 #undef NRL_GN
+}
+
+cudaError_t nrl_parallel_boundary(const float* x_in, const void* embed, int w_f32, const int* tok, const float* o, const float* y,
+                                  const int* slot_of, int top, const float* w1, const float* w2, const float* mu, float eps, float* x_out,
+                                  void* raw, void* h1, void* h2, int h_f32, const int* cu, const int* tok_entry, const int* start,
+                                  const int* state_slot, const float* state, float* carry, const float* commit, float* commit_state, int T,
+                                  int W, cudaStream_t s) {
+  if (T <= 0) return cudaSuccess;
+  const size_t smem = sizeof(float) * 2 * W;
+  if ((x_in == nullptr) == (embed == nullptr) || (embed != nullptr && tok == nullptr) || W < 1 || smem > 200 * 1024 ||
+      (h1 != nullptr && w1 == nullptr) || (h2 != nullptr && w2 == nullptr) || (y != nullptr && (slot_of == nullptr || top < 1)) ||
+      (h1 != nullptr && mu != nullptr && (state == nullptr || carry == nullptr)) || (commit == nullptr) != (commit_state == nullptr) ||
+      (x_out != nullptr && x_out == x_in))
+    return cudaErrorInvalidValue;
+  // tokens per block: one while that fills the GPU, up to eight (the row above a block is read once more per block)
+  const int rows = T >= 8192 ? 8 : T >= 4096 ? 4 : T >= 2048 ? 2 : 1;
+  const ParallelBoundary p = {x_in, embed, tok, o, y, slot_of, top, w1, w2, mu, eps, x_out, raw, h1, h2, cu, tok_entry, start, state_slot,
+                              state, carry, commit, commit_state, T, W, rows};
+  auto ok = [](const void* q, size_t a) { return q == nullptr || aligned(q, a); };
+  const size_t ha = h_f32 ? 16 : 8;
+  const bool vec = W % 4 == 0 && ok(x_in, 16) && ok(o, 16) && ok(y, 16) && ok(w1, 16) && ok(w2, 16) && ok(mu, 16) && ok(x_out, 16) &&
+                   ok(state, 16) && ok(carry, 16) && ok(commit, 16) && ok(commit_state, 16) && ok(raw, ha) && ok(h1, ha) && ok(h2, ha);
+  const int per = vec ? W / 4 : W;
+  const int th = per <= 64 ? 64 : per <= 128 ? 128 : 256;
+  const int blocks = (T + rows - 1) / rows;
+#define NRL_PB(WT_, HT_, V_)                                                                                             \
+  do {                                                                                                                   \
+    auto kern = parallel_boundary_kernel<WT_, HT_, V_>;                                                                  \
+    if (smem > 40 * 1024) {                                                                                              \
+      cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));   \
+      if (e != cudaSuccess) return e;                                                                                    \
+    }                                                                                                                    \
+    kern<<<blocks, th, smem, s>>>(p);                                                                                    \
+    return cudaGetLastError();                                                                                           \
+  } while (0)
+#define NRL_PBV(WT_, HT_)       \
+  do {                          \
+    if (vec) NRL_PB(WT_, HT_, 4); \
+    NRL_PB(WT_, HT_, 1);        \
+  } while (0)
+  if (w_f32 && h_f32) NRL_PBV(float, float);
+  if (w_f32) NRL_PBV(float, __nv_bfloat16);
+  if (h_f32) NRL_PBV(__nv_bfloat16, float);
+  NRL_PBV(__nv_bfloat16, __nv_bfloat16);
+#undef NRL_PBV
+#undef NRL_PB
+}
+
+cudaError_t nrl_gate_cols(const float* in, long si, const float* gate, long sg, float scale, void* out, long so, int out_f32, int T, int C,
+                          cudaStream_t s) {
+  if (T <= 0 || C <= 0) return cudaSuccess;
+  const bool vec = C % 4 == 0 && si % 4 == 0 && sg % 4 == 0 && so % 4 == 0 && aligned(in, 16) && aligned(gate, 16) && aligned(out, out_f32 ? 16 : 8);
+  const int cv = vec ? C / 4 : C;
+  const long n = static_cast<long>(T) * cv;
+  const int blocks = static_cast<int>((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+#define NRL_GC(OT_, V_) gate_cols_kernel<OT_, V_><<<blocks, 256, 0, s>>>(in, si, gate, sg, scale, static_cast<OT_*>(out), so, T, cv)
+  if (out_f32) {
+    if (vec) NRL_GC(float, 4);
+    else NRL_GC(float, 1);
+  } else {
+    if (vec) NRL_GC(__nv_bfloat16, 4);
+    else NRL_GC(__nv_bfloat16, 1);
+  }
+#undef NRL_GC
+  return cudaGetLastError();
 }
 
 cudaError_t nrl_embed_streams(const void* embed, int w_f32, const int* tok, float scale, float* xs, int T, int S, int W, cudaStream_t s) {

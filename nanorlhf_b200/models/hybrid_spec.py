@@ -44,6 +44,7 @@ class MixerSpec:
     # token, plus one rotated key part of `rot_dim` columns shared by the heads; only the latent and that part are cached;
     # `dim` is the unrotated query/key size per head; causal; `head_gate` and `head_sink` as below):
     kv_rank: int = 0
+    q_rank: int = 0              # > 0: queries are projections "uq" of an RMS-normed latent "dq" of that size (weight "dq.norm") instead of "q"
     rot_dim: int = 0             # rotated query/key columns per head, behind the `dim` unrotated ones
     rot_dims: int = 0            # how many of the rot_dim columns turn (the rest pass unchanged)
     rot_base: float = 10000.0    # frequency i of rot_dims / 2 is rot_base^(-2 i / rot_dims)
@@ -66,7 +67,7 @@ class MixerSpec:
                                  # lq2, lk2 [dim]): o = a_1 - lambda a_2 with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, RMS-normed per
                                  # head, times (1 - diff)
     diff: float = 0.0
-    out_gate: bool = False       # the concatenated heads times sigmoid(g h), element by element (tensor "g" [heads * vdim, W])
+    out_gate: bool = False       # (also latent_attention) the concatenated heads times sigmoid(g h), element by element (tensor "g" [heads * vdim, W])
     kv_from: int = -1            # >= 0: no k / v projections; the layer reads the pages of that earlier layer
     # mlstm (matrix memory with exponential gates: log gates i = cap tanh((i h + i.b) / cap), f = logsigmoid(cap tanh((f h + f.b) / cap));
     # m' = max(f + m, i); S = exp(f + m - m') S + exp(i - m') k v^T, n likewise with k; o = S^T q / (max(|n . q|, exp(-m')) + 1e-6) with
@@ -86,6 +87,8 @@ class LayerSpec:
     route: str = "softmax_top"   # "softmax_top": the largest logits (+ bias "router.b"), weights = softmax over the chosen logits
                                  # "softmax_all": scores = softmax over all router outputs, chosen by score + "correction",
                                  #                weights = the chosen scores / their sum * route_scale
+                                 # "sigmoid": scores = sigmoid of the logits, the largest are chosen, weights = the chosen scores
+    weight_input: bool = False   # "softmax_top" / "sigmoid": the weight multiplies the expert's input instead of its result
     route_scale: float = 1.0
     route_groups: int = 1        # "softmax_all": > 1: the router outputs form that many equal groups of neighbours and only experts of the
     route_keep: int = 1          # `route_keep` groups with the largest choice score can be chosen
@@ -109,7 +112,12 @@ class StreamSpec:
     embedding is normed too (tensor "embed.norm").  ``kind`` "hyper": ``streams`` copies of the stream (all equal to the embedding at
     the start); sublayer q of a layer reads ``layernorm(sum_s hc<q>.in[s] x_s)`` (weight norm<q>, bias norm<q>.b) and every stream becomes
     ``x_t <- sum_s hc<q>.mix[s, t] x_s + hc<q>.out[t] y``; the output reads the layer norm of the streams' sum (``hyper_weights`` False:
-    one stream with the plain residual sum, no hc tensors)."""
+    one stream with the plain residual sum, no hc tensors).  ``kind`` "parallel": ``x += mixer(norm1(x)) + ff(norm2(x))``, both of the same
+    x; ``token_shift``: the mixer reads ``h + (h_prev - h) * shift`` with ``h = norm1(x)`` and ``h_prev`` the previous token's h (zeros for the
+    first; tensor "shift").
+
+    ``loop`` (start, stop, times): layers start .. stop - 1 run that many times in a row with the same weights, every pass with cache
+    and state of its own; each pass begins with ``x = loop.in [x; x0]``, x0 the embedding."""
     kind: str = "depth_weighted"
     norm_groups: int = 1
     gated_residual: bool = False
@@ -121,6 +129,9 @@ class StreamSpec:
     logit_scale: float = 1.0
     streams: int = 1                            # "hyper": copies of the residual stream
     hyper_weights: bool = True                  # "hyper": the layers carry hc1 / hc2 tensors
+    token_shift: bool = False                   # "parallel"
+    centred_norm: bool = False                  # "parallel": norm weights are stored around zero (the norm multiplies by 1 + w)
+    loop: Optional[tuple] = None                # "parallel": (start, stop, times)
     tied_head: bool = False                     # logits = embed x (the table itself, without embed_scale); no "head" tensor
 
 
@@ -134,6 +145,7 @@ class TensorModel(nn.Module):
     Subclasses set ``config_class`` (with ``from_pretrained`` / ``to_dict`` / ``layer_specs`` / ``stream_spec`` /
     ``tensor_shapes``) and may override ``free_shape`` (tensors whose shape the config does not fix) and ``init_value``."""
     config_class = None
+    ignore_extra = False                        # tensors the config gives no use for are not read (else they are an error)
     int_tensors = ()                            # names stored as int32
 
     def __init__(self, cfg, shapes: Optional[Dict[str, tuple]] = None, dtype=torch.bfloat16, device="cpu"):
@@ -176,7 +188,7 @@ class TensorModel(nn.Module):
         want = cfg.tensor_shapes()
         missing = [n for n in want if n not in sd]
         extra = [n for n in sd if n not in want]
-        if missing or extra:
+        if missing or (extra and not cls.ignore_extra):
             raise ValueError(f"checkpoint does not fit its config: missing {missing[:4]}, unexpected {extra[:4]}")
         shapes = {n: tuple(sd[n].shape) for n in want}
         for n, shp in want.items():

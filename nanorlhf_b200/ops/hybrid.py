@@ -115,10 +115,11 @@ def group_norm_residual(x, o, gate, gate_bias, w_post, w_pre, groups, eps, h):
     _ext().group_norm_residual(x, o, gate, gate_bias, w_post, w_pre, groups, eps, h)
 
 
-def moe_route(router, router_bias, top, gu=None, ff=0, act=None, ids=None, wts=None):
-    """Top-k routing (softmax over the chosen logits); with ``gu`` / ``act`` also the dense-form expert activations."""
+def moe_route(router, router_bias, top, gu=None, ff=0, act=None, ids=None, wts=None, sigmoid: bool = False, weight_input: bool = False):
+    """Top-k routing, weights = softmax over the chosen logits or (``sigmoid``) each chosen logit's own sigmoid; with ``gu`` / ``act``
+    also the dense-form expert activations (``weight_input``: the weight multiplies the expert's input, not its result)."""
     native._count()
-    _ext().moe_route(router, router_bias, top, gu, ff, act, ids, wts)
+    _ext().moe_route(router, router_bias, top, gu, ff, act, ids, wts, sigmoid, weight_input)
 
 
 def interleave_gate_up(gate, up):
@@ -129,30 +130,38 @@ def interleave_gate_up(gate, up):
     return torch.stack([gate.view(ff // 32, 32, W), up.view(ff // 32, 32, W)], 1).reshape(2 * ff, W)
 
 
-def moe_grouped_ffn(h, ids, wts, w_gate_up, w_down, experts, ff, out, fused_act: bool = False, identity: int = 0):
+def moe_grouped_ffn(h, ids, wts, w_gate_up, w_down, experts, ff, out, fused_act: bool = False, identity: int = 0,
+                    weight_input: bool = False):
     """Expert feed-forwards of a routed batch on the grouped tcgen05 GEMM.  ``h`` bf16 [T, W]; ``ids`` / ``wts`` [T, top] from
     ``moe_route``; ``w_gate_up`` bf16 [experts * 2 ff, W] (per expert its gate rows, then its up rows; ``fused_act``: interleaved
     per 32 features by ``interleave_gate_up``, the SwiGLU is then formed in the GEMM's epilogue); ``w_down`` bf16
     [experts * W, ff]; ``out`` float [T, W] = sum_k wts[t, k] * expert_k(h[t]).  No launch depends on the routing.
     ``identity``: ids ``experts .. experts + identity - 1`` name experts without matrices; their pairs carry weight 0 here and are
-    skipped (the caller adds their share of the input)."""
+    skipped (the caller adds their share of the input).
+    ``weight_input``: the weight multiplies the expert's INPUT: the gate and up products are scaled per row before the activation
+    (the projections have no bias).  ``out`` is then not written; returns ``(y, slot_of)``, the experts' results in expert order and
+    each (token, choice) pair's row, for a boundary kernel that sums them."""
     import torch
     T, W = h.shape
     R = ids.numel()
     ext = _ext()
     native._count(5 if fused_act else 6)
-    slot_of, row_token, _seg, tiles, num_tiles = ext.moe_plan(ids, experts + identity, 128, experts)
+    rw = torch.empty(R, dtype=torch.float32, device=h.device) if weight_input else None
+    slot_of, row_token, _seg, tiles, num_tiles = ext.moe_plan(ids, experts + identity, 128, experts, wts if weight_input else None, rw)
     xp = torch.empty(R, W, dtype=h.dtype, device=h.device)
     ext.gather_rows(h, row_token, xp)
     act = torch.empty(R, ff, dtype=h.dtype, device=h.device)
     if fused_act:
-        ext.gemm_tc_grouped(xp, w_gate_up, None, tiles, num_tiles, 0, act)
+        ext.gemm_tc_grouped(xp, w_gate_up, None, tiles, num_tiles, 0, act, rw)
     else:
         gu = torch.empty(R, 2 * ff, dtype=torch.float32, device=h.device)
         ext.gemm_tc_grouped(xp, w_gate_up, gu, tiles, num_tiles)
-        ext.swiglu_rows(gu, act)
+        ext.swiglu_rows(gu, act, rw)
     y = torch.empty(R, W, dtype=torch.float32, device=h.device)
     ext.gemm_tc_grouped(act, w_down, y, tiles, num_tiles)
+    if weight_input:
+        native._count(-1)
+        return y, slot_of
     ext.moe_combine(y, slot_of, wts, out)
     return out
 
@@ -224,6 +233,29 @@ def rotary_frequencies(dims: int, base: float, scaling=None):
         ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
         out.append(fi / factor * ramp + fi * (1.0 - ramp))
     return out, 0.1 * math.log(factor) + 1.0
+
+
+def parallel_boundary(plan, embed, eps, x_in=None, o=None, y=None, slot_of=None, w1=None, w2=None, mu=None, x_out=None, raw=None, h1=None,
+                      h2=None, state=None, carry=None, commit=None, commit_state=None):
+    """Boundary of a stream whose mixer and feed-forward read the same x: ``x = (x_in or embed[tokens]) + o + sum_k y[slot_of]`` goes to
+    ``x_out`` (float) and ``raw`` (operand type); ``h1 = rmsnorm(x) * w1`` (with ``mu``: moved towards the previous token's row, which an
+    entry's first token finds in its slot of ``state``) and ``h2 = rmsnorm(x) * w2``.  ``carry`` [entries, W] receives the rows that
+    later steps need; the next boundary hands them over (``commit`` -> ``commit_state``)."""
+    native._count()
+    _ext().parallel_boundary(x_in, embed, plan.tokens, o, y, slot_of, w1, w2, mu, eps, x_out, raw, h1, h2, plan.cu, plan.tok_entry,
+                             plan.start, plan.state_slot, state, carry, commit, commit_state)
+
+
+def gate_cols(x, gate, scale, out):
+    """out = scale * x * sigmoid(gate), element by element."""
+    native._count()
+    _ext().gate_cols(x, gate, scale, out)
+
+
+def rmsnorm_cols(x, w, eps, out):
+    """out = x / rms(x) * w over the whole row."""
+    native._count()
+    _ext().gated_part_rmsnorm(x, None, w, x.shape[1], 0, False, eps, 1.0, out)
 
 
 def embed_streams(embed, tok, scale, xs):

@@ -26,6 +26,11 @@ step in a per-sequence slot) and it gives chunked prefill and continuous batchin
   q / k, capped scores, a sink, kept first positions, a bias by distance bucket, values that are the keys, two differential score
   maps, pages borrowed from an earlier layer) and a matrix memory with exponential gates (mLSTM); its router may limit the choice to
   the best groups of experts;
+* a fifth kind, "parallel", adds mixer and feed-forward of the same x, each behind its own norm; the mixer's input may be shifted
+  towards the previous token's (one row per sequence and layer run is carried in the state slot); a range of layers may run several
+  times in a row with shared weights and a projection of [x; embedding] in front of every pass, each pass with pages and state of
+  its own; its latent attention may form queries through a normed latent and gate the heads element by element; its router weighs
+  the experts' inputs with sigmoid scores;
 * the residual stream, its depth-weighted average, norms, scores, softmax, decays and recurrent state are float32 in both
   serving modes; ``dtype="bf16"`` keeps GEMM operands and KV pages in bf16 (fp32 accumulation, fp32 GEMM results),
   ``dtype="fp32"`` keeps everything in float32 with TF32 off;
@@ -34,6 +39,7 @@ step in a per-sequence slot) and it gives chunked prefill and continuous batchin
 """
 from __future__ import annotations
 
+import copy
 import math
 from typing import Dict, List, Optional, Sequence, Tuple
 
@@ -69,7 +75,7 @@ class StepPlan:
 
 class _Mixer:
     __slots__ = ("spec", "cols", "out_col", "out_size", "vec", "k_cache", "v_cache", "conv_state", "state", "w_lr2", "lr_cols", "rank",
-                 "w_uk", "w_uv", "rot_mult", "aux_state", "lam", "owns_kv")
+                 "w_uk", "w_uv", "w_uq", "rot_mult", "aux_state", "lam", "owns_kv")
 
 
 class _Layer:
@@ -78,7 +84,7 @@ class _Layer:
     __slots__ = ("spec", "gain", "dw", "w_in", "w_out", "mixers", "ff_col", "ff_out_col", "n_in", "k_out", "out_pad",
                  "w_pre", "w_post", "gate_col", "gate_bias", "router_col", "router_bias", "w_gate_up", "w_down",
                  "shared_col", "shared_out_col", "sg_col", "side_col", "side_out_col", "side_col0", "hc_in", "hc_out", "hc_mix", "w_pre_b",
-                 "out_bias")
+                 "out_bias", "ff", "shift", "shift_state", "pass_entry")
 
 
 def _pad8(n: int) -> int:
@@ -182,20 +188,61 @@ class HybridSampler:
                     if st.hyper_weights:
                         L.hc_in, L.hc_out, L.hc_mix = (self._f(f"{p}hc{n}.{x}") for x in ("in", "out", "mix"))
                     self.layers.append(L)
+            elif st.kind == "parallel":                   # one stage per layer; its feed-forward reads an operand of its own (L.ff)
+                L = self._build_stage(spec, spec.mixers, False)
+                L.w_pre = self._norm_gain(p + "norm1")
+                L.shift = self._f(p + "shift") if st.token_shift else None
+                if spec.ff:
+                    self._attach_feed_forward(L, spec)
+                    L.ff.w_pre = self._norm_gain(p + "norm2")
+                self.layers.append(L)
             else:
                 raise ValueError(f"unknown stream kind {st.kind!r}")
+        self.w_pass_x = self.w_pass_x0 = None
+        if st.loop:
+            self._unroll_loop(*st.loop)
         self.embed_gain = self._f("embed.norm") if st.kind == "post_norm" else None
         self.side_table = (self._t("side.embed").to(device=dev, dtype=wd).contiguous()
                            if st.kind == "post_norm" and lm.has_tensor("side.embed") else None)
         self.embed = self._t("embed").to(device=dev, dtype=wd).contiguous()
         self.pos_table = self._t("pos").to(device=dev, dtype=wd).contiguous() if st.positions else None
         self.pair_table = self._t("bigram").to(device=dev, dtype=wd).contiguous() if st.pair_buckets else None
-        self.final_gain = self._f("final.norm").reshape(1) if st.kind == "depth_weighted" else self._f("final.norm")
+        self.final_gain = self._f("final.norm").reshape(1) if st.kind == "depth_weighted" else self._norm_gain("final.norm")
         self.final_bias = self._f("final.norm.b") if st.kind == "hyper" and lm.has_tensor("final.norm.b") else None
         V = self.cfg.vocab
         self.head = torch.zeros(_pad8(V), W, dtype=wd, device=dev)
         self.head[:V] = self._t("embed" if st.tied_head else "head").to(device=dev, dtype=wd)
         self._weights_version = self.weights_fingerprint()
+
+    def _norm_gain(self, name):
+        w = self._f(name)
+        return w + 1.0 if self.stream.centred_norm else w
+
+    def _attach_feed_forward(self, L, spec):
+        """Give a parallel layer its feed-forward: own input matrix (it reads another norm), output columns behind the mixer's."""
+        F = self._build_stage(spec, [], True)
+        if F.ff_out_col is not None:
+            F.ff_out_col = (F.ff_out_col[0] + L.k_out, F.ff_out_col[1])
+        L.w_out = torch.cat([L.w_out, F.w_out], 1).contiguous()
+        L.k_out += F.k_out
+        L.out_pad = L.out_pad or F.out_pad
+        F.w_out = None
+        L.ff = F
+
+    def _unroll_loop(self, start: int, stop: int, times: int):
+        """Repeat the layers start .. stop - 1: the runs share their weights, each has pages and state of its own.  The projection in
+        front of a pass is split into its stream half and its embedding half, whose product is formed once per step."""
+        def again(L):
+            c = copy.copy(L)
+            c.mixers = [copy.copy(M) for M in L.mixers]
+            return c
+        body = self.layers[start:stop]
+        passes = [body] + [[again(L) for L in body] for _ in range(times - 1)]
+        for p in passes:
+            p[0].pass_entry = True
+        self.layers = self.layers[:start] + [L for p in passes for L in p] + self.layers[stop:]
+        w, W = self._t("loop.in"), self.cfg.width
+        self.w_pass_x, self.w_pass_x0 = (w[:, c:c + W].to(device=self.device, dtype=self.wdtype).contiguous() for c in (0, W))
 
     def _build_stage(self, spec, mixer_specs, with_ff: bool, gate: Optional[str] = None, side: bool = False) -> _Layer:
         """Fuse every projection that reads the stage's normed input into ``w_in`` and every projection that writes the stream
@@ -208,6 +255,8 @@ class HybridSampler:
         L.w_gate_up = L.w_down = None
         L.shared_col = L.shared_out_col = L.sg_col = L.side_col = L.side_out_col = None
         L.hc_in = L.hc_out = L.hc_mix = L.w_pre_b = L.out_bias = None
+        L.ff = L.shift = L.shift_state = None
+        L.pass_entry = False
         L.side_col0 = 0
         rows_in: List[torch.Tensor] = []
         cols_out: List[torch.Tensor] = []
@@ -240,7 +289,7 @@ class HybridSampler:
         for ms in mixer_specs:
             M = _Mixer()
             M.spec, M.cols, M.vec = ms, {}, {}
-            M.k_cache = M.v_cache = M.conv_state = M.state = M.w_lr2 = M.w_uk = M.w_uv = M.aux_state = None
+            M.k_cache = M.v_cache = M.conv_state = M.state = M.w_lr2 = M.w_uk = M.w_uv = M.w_uq = M.aux_state = None
             M.lam, M.owns_kv = 0.0, True
             q = ms.prefix
             if ms.kind == "window_attention":
@@ -284,9 +333,16 @@ class HybridSampler:
                 for n in ("dt_bias", "A_log", "norm"):
                     M.vec[n] = self._f(q + n)
             elif ms.kind == "latent_attention":
-                for n in ("q", "dkv"):
+                for n in ("dq" if ms.q_rank else "q", "dkv"):
                     M.cols[n] = add_in(q + n)
-                if ms.head_gate:
+                    if ms.q_rank:
+                        pad_in()
+                if ms.q_rank:                              # queries through a latent: its columns padded to whole 16-byte chunks
+                    uq = self._t(q + "uq")
+                    M.w_uq = torch.zeros(_pad8(uq.shape[0]), _pad8(ms.q_rank), dtype=wd, device=dev)
+                    M.w_uq[:uq.shape[0], :ms.q_rank] = uq.to(wd)
+                    M.vec["dq.norm"] = self._f(q + "dq.norm")
+                if ms.head_gate or ms.out_gate:
                     M.cols["g"] = add_in(q + "g")
                 M.vec["dkv.norm"] = self._f(q + "dkv.norm")
                 if ms.head_sink:
@@ -434,11 +490,14 @@ class HybridSampler:
         """Re-fuse the arena when the model's weights changed (the optimizer bumps ``_nrl_version``)."""
         if force or self._weights_version != self.weights_fingerprint():
             pools = [(M.k_cache, M.v_cache, M.conv_state, M.state, M.aux_state) for L in self.layers for M in L.mixers]
+            shifts = [L.shift_state for L in self.layers]
             self._graphs.clear()                          # captured graphs hold the old arena's addresses
             self._graph_seen.clear()
             self._build_arena()
             for M, pl in zip([M for L in self.layers for M in L.mixers], pools):
                 M.k_cache, M.v_cache, M.conv_state, M.state, M.aux_state = pl
+            for L, t in zip(self.layers, shifts):
+                L.shift_state = t
 
     def release(self):
         self._graphs.clear()
@@ -455,6 +514,8 @@ class HybridSampler:
         n = max(1, (pool_tokens + self.PAGE - 1) // self.PAGE)
         f32 = dict(dtype=torch.float32, device=dev)
         for L in self.layers:
+            if L.shift is not None:                        # the last token's normed row of every sequence
+                L.shift_state = torch.zeros(num_slots, self.cfg.width, **f32)
             for M in L.mixers:
                 ms = M.spec
                 if ms.kind == "window_attention":
@@ -570,6 +631,8 @@ class HybridSampler:
             return self._forward_post_norm(plan, rows)
         if self.stream.kind == "hyper":
             return self._forward_hyper(plan, rows)
+        if self.stream.kind == "parallel":
+            return self._forward_parallel(plan, rows)
         return self._forward_depth_weighted(plan, rows)
 
     def _run_mixers(self, L, U, A, plan, eps, ctx=None):
@@ -663,6 +726,60 @@ class HybridSampler:
         hw = h if rows == list(range(T)) else h[torch.tensor(rows, device=dev)]
         return self._mm(hw.contiguous(), self.head)[:, :cfg.vocab]
 
+    def _forward_parallel(self, plan: StepPlan, rows: List[int], keep: Optional[list] = None) -> torch.Tensor:
+        """Mixer and feed-forward side by side on the same x.  One fused kernel per layer boundary adds both results (expert rows are
+        gathered there), forms both norms and the token shift, and hands the shifted rows that later steps need to their slots.
+        ``keep``: a list that receives a copy of the stream after every layer run."""
+        cfg, dev, wd = self.cfg, self.device, self.wdtype
+        T, W, eps = plan.T, cfg.width, cfg.norm_eps
+        f32 = dict(dtype=torch.float32, device=dev)
+        h1 = torch.empty(T, W, dtype=wd, device=dev)
+        h2 = torch.empty(T, W, dtype=wd, device=dev)
+        raw = torch.empty(T, W, dtype=wd, device=dev) if self.stream.loop else None
+        xs = [torch.empty(T, W, **f32), torch.empty(T, W, **f32)]
+        carries = [torch.empty(plan.E, W, **f32), torch.empty(plan.E, W, **f32)] if self.stream.token_shift else None
+        z0 = None                                          # the embedding's half of the projection in front of a pass
+        if self.stream.loop:
+            hy.parallel_boundary(plan, self.embed, eps, raw=raw)
+            z0 = self._mm(raw, self.w_pass_x0)
+        x = o = y = slot_of = None                         # x None: the embedding
+        done = {}                                          # what the last token-shifted boundary left for its state
+        for i, L in enumerate(self.layers):
+            if L.pass_entry:                               # x = loop.in [x; x0], the second half already multiplied
+                if i:                                      # (in front of layer 0 ``raw`` holds the embedding already)
+                    hy.parallel_boundary(plan, self.embed, eps, x_in=x, o=o, y=y, slot_of=slot_of, raw=raw,
+                                         x_out=xs[i & 1] if keep is not None else None, **done)
+                if keep is not None and i:
+                    keep.append(xs[i & 1].clone())
+                x, o, y, slot_of, done = self._mm(raw, self.w_pass_x), z0, None, None, {}
+            F, xn = L.ff, xs[i & 1]
+            carry = carries[i & 1] if L.shift is not None else None
+            hy.parallel_boundary(plan, self.embed, eps, x_in=x, o=o, y=y, slot_of=slot_of, w1=L.w_pre, mu=L.shift, x_out=xn, h1=h1,
+                                 w2=F.w_pre if F is not None else None, h2=h2 if F is not None else None, state=L.shift_state, carry=carry,
+                                 **done)
+            done = dict(commit=carry, commit_state=L.shift_state) if carry is not None else {}
+            if keep is not None and i and not L.pass_entry:
+                keep.append(xn.clone())
+            x, y, slot_of = xn, None, None
+            U = self._mm(h1, L.w_in)                                                  # [T, n_in] float
+            A = (torch.zeros if L.out_pad else torch.empty)(T, L.k_out, dtype=wd, device=dev)
+            self._run_mixers(L, U, A, plan, eps)
+            if F is not None:
+                U = self._mm(h2, F.w_in)
+                if F.ff_col is not None:
+                    self._feed_forward(F, U, A)
+                if F.w_gate_up is not None:
+                    y, slot_of = self._experts_grouped(F, U, h2, None)
+            o = self._mm(A, L.w_out)                                                  # [T, W] float
+        hy.parallel_boundary(plan, self.embed, eps, x_in=x, o=o, y=y, slot_of=slot_of, w1=self.final_gain, h1=h1,
+                             x_out=xs[len(self.layers) & 1] if keep is not None else None, **done)
+        if keep is not None:
+            keep.append(xs[len(self.layers) & 1].clone())
+        if not rows:
+            return torch.empty(0, cfg.vocab, **f32)
+        hw = h1 if rows == list(range(T)) else h1[torch.tensor(rows, device=dev)]
+        return self._mm(hw.contiguous(), self.head)[:, :cfg.vocab]
+
     def _rot_attention(self, M, U, plan, eps, out):
         """Attention with rotated (or plain) grouped heads and the optional terms of its spec.  One launch finishes the queries in
         place (bias, rotation, unit norm) and writes keys and values to their pages; the paged kernel applies cap, distance bias,
@@ -712,14 +829,23 @@ class HybridSampler:
     def _latent_attention(self, M, U, plan, eps, out):
         """Latent attention in its absorbed form.  The cache holds one row [latent | rotated shared key part] per token; a head's
         query is taken into that space (``uk_h^T q_unrotated | q_rotated``), the paged kernel treats the row as the one key head
-        whose first ``kv_rank`` columns are also the value, and the latent result is expanded by ``uv_h`` afterwards; the gate and the
-        sink are per head, so they commute with the expansion."""
+        whose first ``kv_rank`` columns are also the value, and the latent result is expanded by ``uv_h`` afterwards; a gate and a
+        sink per head commute with the expansion, an element-wise gate follows it.  Queries may come through a normed latent of
+        their own (``q_rank``)."""
         ms = M.spec
         T, dev, wd = plan.T, U.device, self.wdtype
         H, dn, dr, r, dv = ms.heads, ms.dim, ms.rot_dim, ms.kv_rank, ms.vdim
-        (cq, nq), (cd, nd) = M.cols["q"], M.cols["dkv"]
+        cd, nd = M.cols["dkv"]
         D = r + dr
-        q = U[:, cq:cq + nq]
+        if ms.q_rank:
+            cq, nq = M.cols["dq"]
+            kq = M.w_uq.shape[1]
+            c_q = (torch.zeros if kq != nq else torch.empty)(T, kq, dtype=wd, device=dev)
+            hy.rmsnorm_cols(U[:, cq:cq + nq], M.vec["dq.norm"], eps, c_q[:, :nq])
+            q = self._mm(c_q, M.w_uq)[:, :H * (dn + dr)]
+        else:
+            cq, nq = M.cols["q"]
+            q = U[:, cq:cq + nq]
         # queries head-major [H, T, D]: the batched GEMM writes a head's absorbed columns in place, the kernel its rotated ones
         qa = torch.empty(H, T, D, dtype=torch.float32, device=dev)
         if self.fp32:
@@ -741,6 +867,17 @@ class HybridSampler:
         lat = torch.empty(T, H * r, dtype=wd, device=dev)
         hy.window_attention(qa, M.k_cache, M.k_cache, plan, 1 << 30, ms.scale, ms.out_scale, lat, gate=gate, head_sink=M.vec.get("sink"),
                             value_size=r)
+        if ms.out_gate:
+            cg, ng = M.cols["g"]
+            heads = torch.empty(T, H * dv, dtype=torch.float32, device=dev)
+            native._count()
+            dst = heads.unflatten(1, (H, dv)).transpose(0, 1)
+            if self.fp32:
+                torch.bmm(lat.unflatten(1, (H, r)).transpose(0, 1), M.w_uv, out=dst)
+            else:
+                torch.bmm(lat.unflatten(1, (H, r)).transpose(0, 1), M.w_uv, out_dtype=torch.float32, out=dst)
+            hy.gate_cols(heads, U[:, cg:cg + ng], 1.0, out)
+            return
         # expansion per head straight into the out-projection's operand (float32 accumulation, rounded once)
         native._count()
         torch.bmm(lat.unflatten(1, (H, r)).transpose(0, 1), M.w_uv, out=out.unflatten(1, (H, dv)).transpose(0, 1))
@@ -814,7 +951,8 @@ class HybridSampler:
 
     def _experts_grouped(self, L, U, h, o, want_self: bool = False):
         """Route, then run only the chosen experts: rows sorted by expert through two grouped GEMMs.  ``want_self``: also return the
-        per-token weight of the chosen identity experts (None without such experts)."""
+        per-token weight of the chosen identity experts (None without such experts).  Experts whose input is weighed return their
+        rows in expert order and every (token, choice) pair's row instead of the sum."""
         spec = L.spec
         T, dev = h.shape[0], h.device
         rc, E = L.router_col
@@ -827,7 +965,10 @@ class HybridSampler:
             hy.moe_route_all(U[:, rc:rc + E], L.router_bias, spec.experts, spec.top, spec.route_scale, ids=ids, wts=wts, self_w=self_w,
                              groups=spec.route_groups, keep=spec.route_keep)
         else:
-            hy.moe_route(U[:, rc:rc + E], L.router_bias, spec.top, ids=ids, wts=wts)
+            hy.moe_route(U[:, rc:rc + E], L.router_bias, spec.top, ids=ids, wts=wts, sigmoid=spec.route == "sigmoid")
+        if spec.weight_input:                              # the weights are spent inside: what is left is a sum of rows
+            return hy.moe_grouped_ffn(h, ids, wts, L.w_gate_up, L.w_down, spec.experts, spec.ff, None, fused_act=spec.ff % 32 == 0,
+                                      weight_input=True)
         y = torch.empty(T, self.cfg.width, dtype=torch.float32, device=dev)
         hy.moe_grouped_ffn(h, ids, wts, L.w_gate_up, L.w_down, spec.experts, spec.ff, y, fused_act=spec.ff % 32 == 0,
                            identity=spec.identity_experts)
@@ -848,7 +989,8 @@ class HybridSampler:
             return self_w
         if spec.ff_kind == "moe":
             rc, E = L.router_col
-            hy.moe_route(U[:, rc:rc + E], L.router_bias, spec.top, gu=U[:, c:c + n], ff=spec.ff, act=A[:, oc:oc + on])
+            hy.moe_route(U[:, rc:rc + E], L.router_bias, spec.top, gu=U[:, c:c + n], ff=spec.ff, act=A[:, oc:oc + on],
+                         sigmoid=spec.route == "sigmoid", weight_input=spec.weight_input)
         elif spec.ff_act == "swiglu":
             hy.swiglu_cols(U[:, c:c + n], None, A[:, oc:oc + on])
         else:
