@@ -1,7 +1,7 @@
 """Serving throughput of the hybrid step engine (Nezavik) beside the paged-KV transformer engine (Qwen2) at equal size,
 plus each new kernel against its roofline and against the like kernel of the transformer path; with ``--serve-model vilosun``
 the Vilosun family beside Nezavik (same engine) at equal size, and the kernels it adds beside Nezavik's like kernels; with
-``--serve-model damilix`` the Damilix family beside Vilosun in the same way, ``--serve-model lukarax`` the Lukarax family beside Damilix.
+``--serve-model damilix`` the Damilix family beside Vilosun in the same way, ``--serve-model lukarax`` the Lukarax family and ``--serve-model lopovik`` the Lopovik family beside Damilix.
 
 Run through ``python bench.py --serve-bench`` (one GPU).  Random weights, synthetic token ids.  End-to-end numbers go
 through the engines' public ``generate`` (two runs that differ by `new` generated tokens: the difference is `new` decode steps,
@@ -727,10 +727,180 @@ def kernels(width=2048, batch=16, prompt_len=2048, window=1024, decode_batch=256
     return out
 
 
+def lopovik_config(width: int, n_runs: int, vocab: int, experts: int = 16, top: int = 2, kv_rank: int = 256, rot_dim: int = 64, times: int = 2):
+    """Heads and latent as in ``damilix_config`` with queries through a latent of half the width; feed-forwards alternate between a dense
+    one of 4 x width and `experts` experts of which `top` hold as many weights.  ``n_runs`` layer RUNS (the depth that is computed): the
+    middle half of them is one block of layers run ``times`` times."""
+    from nanorlhf_b200.models.lopovik import LopovikConfig
+    H = width // 128
+    ff = max(128, (8 * width // (3 * top) + 127) // 128 * 128)
+    mixer = {"heads": H, "dim": 128, "rot_dim": rot_dim, "vdim": 128, "kv_rank": kv_rank, "q_rank": width // 2,
+             "scale": (128 + rot_dim) ** -0.5, "rot": {"base": 1e6, "dims": rot_dim}}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    looped = n_runs // 2 // times
+    n = n_runs - looped * (times - 1)
+    start = (n - looped) // 2
+    layers = [{"type": "latent_attention", "mixer": mixer, "mlp": moe if i % 2 else {"kind": "dense", "ff": 4 * width}} for i in range(n)]
+    return LopovikConfig.from_dict({"architecture": "Lopovik", "layers": layers, "loop": {"start": start, "stop": start + looped, "times": times},
+                                    "norm": {"eps": 1e-6}, "vocab": vocab, "width": width})
+
+
+def end_to_end_lopovik(width, n_runs, batch, prompt_len, new=128, vocab=32768):
+    """Lopovik beside Damilix (the closest family: same engine, latent attention, routed experts) at equal width and computed depth."""
+    from nanorlhf_b200.models.damilix import DamilixForCausalLM
+    from nanorlhf_b200.models.lopovik import LopovikForCausalLM
+    from nanorlhf_b200.sampler.hybrid_sampler import HybridSampler
+    dev = torch.device("cuda:0")
+    g = torch.Generator().manual_seed(0)
+    prompts = torch.randint(0, vocab - 2, (batch, prompt_len), generator=g).tolist()
+    res = {"width": width, "layer_runs": n_runs, "batch": batch, "prompt_len": prompt_len, "new_tokens": new}
+    for name, make in (("lopovik", lambda: LopovikForCausalLM.from_config(lopovik_config(width, n_runs, vocab), torch.bfloat16, dev, seed=0)),
+                       ("damilix", lambda: DamilixForCausalLM.from_config(damilix_config(width, n_runs, vocab), torch.bfloat16, dev, seed=0, gla_rank=64))):
+        model = make()
+        eng = HybridSampler(model, dtype="bf16", max_num_seqs=batch, prefill_token_budget=16384)
+        pre, step = _gen_times(lambda p, mt: eng.generate(p, 1, 1.0, 1.0, mt, None, vocab - 1, 1), prompts, new)
+        res[name] = {"params_m": round(sum(p.numel() for p in model.parameters()) / 1e6, 1),
+                     "prefill_tok_s": round(batch * prompt_len / pre), "decode_tok_s": round(batch / step),
+                     "decode_ms_per_step": round(step * 1e3, 3)}
+        eng.release()
+        del eng, model
+        torch.cuda.empty_cache()
+    return res
+
+
+def kernels_lopovik(width=2048, batch=16, prompt_len=2048, decode_batch=256, ctx=2048, experts=16, top=2, kv_rank=256, rot_dim=64):
+    """The kernels Lopovik adds to the step engine, each beside the like kernel of the Damilix / Vilosun / Nezavik paths."""
+    from nanorlhf_b200 import _C
+    from nanorlhf_b200.ops import gemm as _gemm, hybrid as hy
+    from nanorlhf_b200.sampler.hybrid_sampler import StepPlan
+    hbm, flops_peak, which = _peaks()
+    dev = torch.device("cuda:0")
+    out = {"roofline": which, "width": width}
+    H, DL, qr = width // 128, kv_rank + rot_dim, width // 2
+    ff = max(128, (8 * width // (3 * top) + 127) // 128 * 128)
+    bf = torch.bfloat16
+
+    def plan_for(B, n_new, n_old):
+        s = _C.StepScheduler((n_old + n_new + 15) // 16 * B + 8, 16, B)
+        sids = [s.open() for _ in range(B)]
+        if n_old:
+            s.plan(sids, [n_old] * B)
+        data, E, T, MB = s.plan(sids, [n_new] * B)
+        return StepPlan(torch.from_numpy(data).to(dev), E, T, MB), s
+
+    def report(name, sec, bytes_, flops=0.0):
+        floor = max(bytes_ / hbm, flops / flops_peak)
+        out[name] = {"us": round(sec * 1e6, 1), "gb_s": round(bytes_ / sec / 1e9, 1), "tflop_s": round(flops / sec / 1e12, 2),
+                     "roofline_frac": round(floor / sec, 3)}
+
+    for phase, B, n_new, n_old in (("prefill", batch, prompt_len, 0), ("decode", decode_batch, 1, ctx - 1)):
+        plan, sched = plan_for(B, n_new, n_old)
+        T = plan.T
+        f32 = dict(dtype=torch.float32, device=dev)
+        plan.tokens.copy_(torch.randint(0, 32000, (T,), dtype=torch.int32, device=dev))
+        emb = torch.randn(32768, width, device=dev).bfloat16()
+        # -- layer boundary: residual add, two norms, token shift (and the gathered expert rows) vs one norm of one sublayer's result
+        x, o, xn = torch.randn(T, width, **f32), torch.randn(T, width, **f32), torch.empty(T, width, **f32)
+        h1, h2 = torch.empty(T, width, dtype=bf, device=dev), torch.empty(T, width, dtype=bf, device=dev)
+        w1, w2, mu = torch.ones(width, **f32), torch.ones(width, **f32), torch.full((width,), 0.3, **f32)
+        state, carry, old = torch.zeros(B, width, **f32), torch.empty(B, width, **f32), torch.zeros(B, width, **f32)
+        args = dict(x_in=x, o=o, w1=w1, w2=w2, mu=mu, x_out=xn, h1=h1, h2=h2, state=state, carry=carry, commit=carry.clone(), commit_state=old)
+        sec = _time(lambda: hy.parallel_boundary(plan, emb, 1e-6, **args))
+        report(f"{phase}.parallel_boundary", sec, T * width * (4.0 * 3 + 2 * 2) + B * width * 16.0)
+        y, slot_of = torch.randn(T * top, width, **f32), torch.randperm(T * top, device=dev).int()
+        sec = _time(lambda: hy.parallel_boundary(plan, emb, 1e-6, y=y, slot_of=slot_of, **args))
+        report(f"{phase}.parallel_boundary(+ {top} expert rows)", sec, T * width * (4.0 * (3 + top) + 2 * 2) + B * width * 16.0)
+        sec = _time(lambda: hy.parallel_boundary(plan, emb, 1e-6, x_in=x, o=o, raw=h1))
+        report(f"{phase}.parallel_boundary(in front of a pass)", sec, T * width * (4.0 * 2 + 2))
+        sw = torch.rand(T, **f32)
+        sec = _time(lambda: hy.post_norm_residual(x, o, sw, w1, None, 1e-6, h1))
+        report(f"{phase}.damilix.post_norm_residual", sec, T * width * (4.0 * 3 + 2))
+        del y, xn
+        # -- query latent: norm of the latent columns, then the second projection; element-wise output gate
+        n_in = qr + DL + H * 128
+        U = torch.randn(T, n_in, **f32)
+        cq, dqw = torch.empty(T, qr, dtype=bf, device=dev), torch.ones(qr, **f32)
+        sec = _time(lambda: hy.rmsnorm_cols(U[:, :qr], dqw, 1e-6, cq))
+        report(f"{phase}.rmsnorm_cols(query latent {qr})", sec, T * qr * 6.0)
+        heads, gated = torch.randn(T, H * 128, **f32), torch.empty(T, H * 128, dtype=bf, device=dev)
+        sec = _time(lambda: hy.gate_cols(heads, U[:, qr + DL:], 1.0, gated))
+        report(f"{phase}.gate_cols", sec, T * H * 128 * 10.0)
+        sec = _time(lambda: hy.gated_part_rmsnorm(heads, U[:, qr + DL:], torch.ones(128, **f32), 128, "silu", False, 1e-6, 1.0, gated))
+        report(f"{phase}.damilix.gated_part_rmsnorm", sec, T * H * 128 * 10.0)
+        wuq = (torch.randn(H * (128 + rot_dim), qr, device=dev) * qr ** -0.5).bfloat16()
+        q = torch.empty(T, H * (128 + rot_dim), **f32)
+        sec = _time(lambda: _gemm.gemm(cq, wuq, out_f32=q))
+        report(f"{phase}.query_projection(gemm, K {qr})", sec, T * (qr * 2.0 + q.shape[1] * 4.0) + wuq.numel() * 2.0, flops=2.0 * T * wuq.numel())
+        wq = (torch.randn(H * (128 + rot_dim), width, device=dev) * width ** -0.5).bfloat16()
+        sec = _time(lambda: _gemm.gemm(h1, wq, out_f32=q))
+        report(f"{phase}.damilix.query_projection(gemm, K {width})", sec, T * (width * 2.0 + q.shape[1] * 4.0) + wq.numel() * 2.0,
+               flops=2.0 * T * wq.numel())
+        # -- projection in front of a pass (the stream's half)
+        wp = (torch.randn(width, width, device=dev) * width ** -0.5).bfloat16()
+        sec = _time(lambda: _gemm.gemm(h1, wp, out_f32=x))
+        report(f"{phase}.pass_projection(gemm)", sec, T * width * 6.0 + wp.numel() * 2.0, flops=2.0 * T * wp.numel())
+        # -- cache write, attention without / with the gate per head, expansion per head
+        dkv, nw = U[:, qr:qr + DL], torch.ones(kv_rank, **f32)
+        freq = torch.tensor(hy.rotary_frequencies(rot_dim, 1e6)[0], dtype=torch.float64, device=dev)
+        n_pages = sched.num_free_blocks() + plan.max_blocks * B + 8
+        lc = torch.randn(n_pages, 1, 16, DL, device=dev).bfloat16()
+        qa, qn = torch.randn(H, T, DL, **f32), torch.empty(H, T, 128, dtype=bf, device=dev)
+        sec = _time(lambda: hy.latent_kv_write(q, H, 128, rot_dim, dkv, nw, 1e-6, freq, rot_dim, 1.0, True, plan, lc, qa, qn))
+        report(f"{phase}.latent_kv_write", sec, T * (DL * 6.0 + H * (rot_dim * 8.0 + 128 * 6.0)))
+        sink, hg = torch.randn(H, **f32), torch.randn(T, H, **f32)
+        lat = torch.empty(T, H * kv_rank, dtype=bf, device=dev)
+        keys = (sum(p + 1 for p in range(n_new)) if phase == "prefill" else ctx) * B
+        byt = (T * H * DL * 4.0 + T * H * kv_rank * 2.0 + T * DL * 2.0) if phase == "prefill" else (keys * DL * 2.0 + T * H * (DL * 4.0 + kv_rank * 2.0))
+        it, wm = (3, 1) if phase == "prefill" else (20, 5)
+        sec = _time(lambda: hy.window_attention(qa, lc, lc, plan, 1 << 30, 0.07, 1.0, lat, head_sink=sink, value_size=kv_rank), iters=it, warm=wm)
+        report(f"{phase}.latent_attention(row {DL}, value {kv_rank})", sec, byt, flops=2.0 * keys * H * (DL + kv_rank))
+        sec = _time(lambda: hy.window_attention(qa, lc, lc, plan, 1 << 30, 0.07, 1.0, lat, gate=hg, head_sink=sink, value_size=kv_rank), iters=it, warm=wm)
+        report(f"{phase}.damilix.latent_attention(gate per head)", sec, byt, flops=2.0 * keys * H * (DL + kv_rank))
+        wuv = (torch.randn(H, kv_rank, 128, device=dev) * kv_rank ** -0.5).bfloat16()
+        lt = lat.unflatten(1, (H, kv_rank)).transpose(0, 1)
+        sec = _time(lambda: torch.bmm(lt, wuv, out_dtype=torch.float32, out=heads.unflatten(1, (H, 128)).transpose(0, 1)))
+        report(f"{phase}.expansion(batched, float result)", sec, T * H * (kv_rank * 2.0 + 128 * 4.0), flops=2.0 * T * H * kv_rank * 128)
+        sec = _time(lambda: torch.bmm(lt, wuv, out=gated.unflatten(1, (H, 128)).transpose(0, 1)))
+        report(f"{phase}.damilix.expansion(batched, bf16 result)", sec, T * H * (kv_rank * 2.0 + 128 * 2.0), flops=2.0 * T * H * kv_rank * 128)
+        del lc, qa, qn, lat, lt, q, heads, gated, U
+        # -- routing and experts: sigmoid scores on the input vs softmax scores on the result (+ the sum over the chosen)
+        zr = torch.randn(T, experts + 2, **f32)
+        ids, wts = torch.empty(T, top, dtype=torch.int32, device=dev), torch.empty(T, top, **f32)
+        sec = _time(lambda: hy.moe_route_all(zr, None, experts + 2, top, 1.5, ids=ids, wts=wts))
+        report(f"{phase}.damilix.moe_route_all", sec, T * ((experts + 2) * 4.0 + top * 8.0))
+        z = zr[:, :experts]
+        sec = _time(lambda: hy.moe_route(z, None, top, ids=ids, wts=wts, sigmoid=True))
+        report(f"{phase}.moe_route(sigmoid)", sec, T * (experts * 4.0 + top * 8.0))
+        wg = (torch.randn(experts * 2 * ff, width, device=dev) * width ** -0.5).bfloat16()
+        wd = (torch.randn(experts * width, ff, device=dev) * ff ** -0.5).bfloat16()
+        res = torch.empty(T, width, **f32)
+        wbytes = min(experts, T * top) * 3.0 * ff * width * 2.0
+        fl = 6.0 * T * top * width * ff
+        it, wm = (5, 2) if phase == "prefill" else (20, 5)
+        sec = _time(lambda: hy.moe_grouped_ffn(h2, ids, wts, wg, wd, experts, ff, None, fused_act=True, weight_input=True), iters=it, warm=wm)
+        report(f"{phase}.moe_grouped_ffn(weights on the input)", sec, wbytes + T * width * (2.0 + 4.0 * top), flops=fl)
+        sec = _time(lambda: hy.moe_grouped_ffn(h2, ids, wts, wg, wd, experts, ff, res, fused_act=True), iters=it, warm=wm)
+        report(f"{phase}.damilix.moe_grouped_ffn(weights on the result)", sec, wbytes + T * width * 6.0, flops=fl)
+        del wg, wd
+    return out
+
+
 def main(quick: bool = False, small: bool = False, model: str = "nezavik"):
     from nanorlhf_b200.ops import native
     global SMALL
     native.load()
+    if model == "lopovik":
+        SMALL = small
+        if small:
+            print(json.dumps({"bench": "serve-lopovik-small",
+                              "kernels": kernels_lopovik(width=1024, batch=8, prompt_len=1024, decode_batch=64, ctx=1024)}))
+            return None
+        res = {"bench": "serve-lopovik", "kernels": kernels_lopovik(), "end_to_end": []}
+        for width, runs, batch, plen in ((1024, 8, 32, 1024), (2048, 8, 16, 2048)) if not quick else ((1024, 4, 8, 512),):
+            res["end_to_end"].append(end_to_end_lopovik(width, runs, batch, plen))
+        res["gpu_launches"] = native.launches()
+        print(json.dumps(res))
+        return res
     if model == "lukarax":
         SMALL = small
         if small:
@@ -781,4 +951,4 @@ def main(quick: bool = False, small: bool = False, model: str = "nezavik"):
 
 if __name__ == "__main__":
     main(quick="--quick" in sys.argv, small="--small" in sys.argv,
-         model="lukarax" if "--lukarax" in sys.argv else "damilix" if "--damilix" in sys.argv else "vilosun" if "--vilosun" in sys.argv else "nezavik")
+         model="lopovik" if "--lopovik" in sys.argv else "lukarax" if "--lukarax" in sys.argv else "damilix" if "--damilix" in sys.argv else "vilosun" if "--vilosun" in sys.argv else "nezavik")
