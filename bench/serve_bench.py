@@ -46,6 +46,23 @@ def _time(fn, iters=10, warm=3):
     return e0.elapsed_time(e1) / iters * 1e-3          # seconds
 
 
+def _time_graphed(fn, reps=20, warm=3):
+    """Seconds per call of a short kernel inside a CUDA graph of ``reps`` calls (decode steps are replayed as graphs: a launch from the
+    host, which takes longer than such a kernel, is not part of them).  Inputs stay in L2, as a decode step's activations do."""
+    if SMALL:
+        return _time(fn)
+    for _ in range(warm):
+        fn()
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        for _ in range(reps):
+            fn()
+    sec = _time(g.replay, iters=5, warm=2) / reps
+    del g
+    return sec
+
+
 def nezavik_config(width: int, n_layers: int, vocab: int, window: int = 1024, max_positions: int = 8192):
     from nanorlhf_b200.models.nezavik import NezavikConfig
     H = width // 128
@@ -796,6 +813,7 @@ def kernels_lopovik(width=2048, batch=16, prompt_len=2048, decode_batch=256, ctx
     for phase, B, n_new, n_old in (("prefill", batch, prompt_len, 0), ("decode", decode_batch, 1, ctx - 1)):
         plan, sched = plan_for(B, n_new, n_old)
         T = plan.T
+        tm = _time_graphed if phase == "decode" else _time
         f32 = dict(dtype=torch.float32, device=dev)
         plan.tokens.copy_(torch.randint(0, 32000, (T,), dtype=torch.int32, device=dev))
         emb = torch.randn(32768, width, device=dev).bfloat16()
@@ -805,39 +823,40 @@ def kernels_lopovik(width=2048, batch=16, prompt_len=2048, decode_batch=256, ctx
         w1, w2, mu = torch.ones(width, **f32), torch.ones(width, **f32), torch.full((width,), 0.3, **f32)
         state, carry, old = torch.zeros(B, width, **f32), torch.empty(B, width, **f32), torch.zeros(B, width, **f32)
         args = dict(x_in=x, o=o, w1=w1, w2=w2, mu=mu, x_out=xn, h1=h1, h2=h2, state=state, carry=carry, commit=carry.clone(), commit_state=old)
-        sec = _time(lambda: hy.parallel_boundary(plan, emb, 1e-6, **args))
+        sec = tm(lambda: hy.parallel_boundary(plan, emb, 1e-6, **args))
         report(f"{phase}.parallel_boundary", sec, T * width * (4.0 * 3 + 2 * 2) + B * width * 16.0)
         y, slot_of = torch.randn(T * top, width, **f32), torch.randperm(T * top, device=dev).int()
-        sec = _time(lambda: hy.parallel_boundary(plan, emb, 1e-6, y=y, slot_of=slot_of, **args))
+        sec = tm(lambda: hy.parallel_boundary(plan, emb, 1e-6, y=y, slot_of=slot_of, **args))
         report(f"{phase}.parallel_boundary(+ {top} expert rows)", sec, T * width * (4.0 * (3 + top) + 2 * 2) + B * width * 16.0)
-        sec = _time(lambda: hy.parallel_boundary(plan, emb, 1e-6, x_in=x, o=o, raw=h1))
+        sec = tm(lambda: hy.parallel_boundary(plan, emb, 1e-6, x_in=x, o=o, raw=h1))
         report(f"{phase}.parallel_boundary(in front of a pass)", sec, T * width * (4.0 * 2 + 2))
         sw = torch.rand(T, **f32)
-        sec = _time(lambda: hy.post_norm_residual(x, o, sw, w1, None, 1e-6, h1))
+        sec = tm(lambda: hy.post_norm_residual(x, o, sw, w1, None, 1e-6, h1))
         report(f"{phase}.damilix.post_norm_residual", sec, T * width * (4.0 * 3 + 2))
         del y, xn
         # -- query latent: norm of the latent columns, then the second projection; element-wise output gate
         n_in = qr + DL + H * 128
         U = torch.randn(T, n_in, **f32)
         cq, dqw = torch.empty(T, qr, dtype=bf, device=dev), torch.ones(qr, **f32)
-        sec = _time(lambda: hy.rmsnorm_cols(U[:, :qr], dqw, 1e-6, cq))
+        sec = tm(lambda: hy.rmsnorm_cols(U[:, :qr], dqw, 1e-6, cq))
         report(f"{phase}.rmsnorm_cols(query latent {qr})", sec, T * qr * 6.0)
         heads, gated = torch.randn(T, H * 128, **f32), torch.empty(T, H * 128, dtype=bf, device=dev)
-        sec = _time(lambda: hy.gate_cols(heads, U[:, qr + DL:], 1.0, gated))
+        sec = tm(lambda: hy.gate_cols(heads, U[:, qr + DL:], 1.0, gated))
         report(f"{phase}.gate_cols", sec, T * H * 128 * 10.0)
-        sec = _time(lambda: hy.gated_part_rmsnorm(heads, U[:, qr + DL:], torch.ones(128, **f32), 128, "silu", False, 1e-6, 1.0, gated))
+        ones = torch.ones(128, **f32)
+        sec = tm(lambda: hy.gated_part_rmsnorm(heads, U[:, qr + DL:], ones, 128, "silu", False, 1e-6, 1.0, gated))
         report(f"{phase}.damilix.gated_part_rmsnorm", sec, T * H * 128 * 10.0)
         wuq = (torch.randn(H * (128 + rot_dim), qr, device=dev) * qr ** -0.5).bfloat16()
         q = torch.empty(T, H * (128 + rot_dim), **f32)
-        sec = _time(lambda: _gemm.gemm(cq, wuq, out_f32=q))
+        sec = tm(lambda: _gemm.gemm(cq, wuq, out_f32=q))
         report(f"{phase}.query_projection(gemm, K {qr})", sec, T * (qr * 2.0 + q.shape[1] * 4.0) + wuq.numel() * 2.0, flops=2.0 * T * wuq.numel())
         wq = (torch.randn(H * (128 + rot_dim), width, device=dev) * width ** -0.5).bfloat16()
-        sec = _time(lambda: _gemm.gemm(h1, wq, out_f32=q))
+        sec = tm(lambda: _gemm.gemm(h1, wq, out_f32=q))
         report(f"{phase}.damilix.query_projection(gemm, K {width})", sec, T * (width * 2.0 + q.shape[1] * 4.0) + wq.numel() * 2.0,
                flops=2.0 * T * wq.numel())
         # -- projection in front of a pass (the stream's half)
         wp = (torch.randn(width, width, device=dev) * width ** -0.5).bfloat16()
-        sec = _time(lambda: _gemm.gemm(h1, wp, out_f32=x))
+        sec = tm(lambda: _gemm.gemm(h1, wp, out_f32=x))
         report(f"{phase}.pass_projection(gemm)", sec, T * width * 6.0 + wp.numel() * 2.0, flops=2.0 * T * wp.numel())
         # -- cache write, attention without / with the gate per head, expansion per head
         dkv, nw = U[:, qr:qr + DL], torch.ones(kv_rank, **f32)
@@ -845,41 +864,39 @@ def kernels_lopovik(width=2048, batch=16, prompt_len=2048, decode_batch=256, ctx
         n_pages = sched.num_free_blocks() + plan.max_blocks * B + 8
         lc = torch.randn(n_pages, 1, 16, DL, device=dev).bfloat16()
         qa, qn = torch.randn(H, T, DL, **f32), torch.empty(H, T, 128, dtype=bf, device=dev)
-        sec = _time(lambda: hy.latent_kv_write(q, H, 128, rot_dim, dkv, nw, 1e-6, freq, rot_dim, 1.0, True, plan, lc, qa, qn))
+        sec = tm(lambda: hy.latent_kv_write(q, H, 128, rot_dim, dkv, nw, 1e-6, freq, rot_dim, 1.0, True, plan, lc, qa, qn))
         report(f"{phase}.latent_kv_write", sec, T * (DL * 6.0 + H * (rot_dim * 8.0 + 128 * 6.0)))
         sink, hg = torch.randn(H, **f32), torch.randn(T, H, **f32)
         lat = torch.empty(T, H * kv_rank, dtype=bf, device=dev)
         keys = (sum(p + 1 for p in range(n_new)) if phase == "prefill" else ctx) * B
         byt = (T * H * DL * 4.0 + T * H * kv_rank * 2.0 + T * DL * 2.0) if phase == "prefill" else (keys * DL * 2.0 + T * H * (DL * 4.0 + kv_rank * 2.0))
-        it, wm = (3, 1) if phase == "prefill" else (20, 5)
-        sec = _time(lambda: hy.window_attention(qa, lc, lc, plan, 1 << 30, 0.07, 1.0, lat, head_sink=sink, value_size=kv_rank), iters=it, warm=wm)
+        sec = tm(lambda: hy.window_attention(qa, lc, lc, plan, 1 << 30, 0.07, 1.0, lat, head_sink=sink, value_size=kv_rank))
         report(f"{phase}.latent_attention(row {DL}, value {kv_rank})", sec, byt, flops=2.0 * keys * H * (DL + kv_rank))
-        sec = _time(lambda: hy.window_attention(qa, lc, lc, plan, 1 << 30, 0.07, 1.0, lat, gate=hg, head_sink=sink, value_size=kv_rank), iters=it, warm=wm)
+        sec = tm(lambda: hy.window_attention(qa, lc, lc, plan, 1 << 30, 0.07, 1.0, lat, gate=hg, head_sink=sink, value_size=kv_rank))
         report(f"{phase}.damilix.latent_attention(gate per head)", sec, byt, flops=2.0 * keys * H * (DL + kv_rank))
         wuv = (torch.randn(H, kv_rank, 128, device=dev) * kv_rank ** -0.5).bfloat16()
         lt = lat.unflatten(1, (H, kv_rank)).transpose(0, 1)
-        sec = _time(lambda: torch.bmm(lt, wuv, out_dtype=torch.float32, out=heads.unflatten(1, (H, 128)).transpose(0, 1)))
+        sec = tm(lambda: torch.bmm(lt, wuv, out_dtype=torch.float32, out=heads.unflatten(1, (H, 128)).transpose(0, 1)))
         report(f"{phase}.expansion(batched, float result)", sec, T * H * (kv_rank * 2.0 + 128 * 4.0), flops=2.0 * T * H * kv_rank * 128)
-        sec = _time(lambda: torch.bmm(lt, wuv, out=gated.unflatten(1, (H, 128)).transpose(0, 1)))
+        sec = tm(lambda: torch.bmm(lt, wuv, out=gated.unflatten(1, (H, 128)).transpose(0, 1)))
         report(f"{phase}.damilix.expansion(batched, bf16 result)", sec, T * H * (kv_rank * 2.0 + 128 * 2.0), flops=2.0 * T * H * kv_rank * 128)
         del lc, qa, qn, lat, lt, q, heads, gated, U
         # -- routing and experts: sigmoid scores on the input vs softmax scores on the result (+ the sum over the chosen)
         zr = torch.randn(T, experts + 2, **f32)
         ids, wts = torch.empty(T, top, dtype=torch.int32, device=dev), torch.empty(T, top, **f32)
-        sec = _time(lambda: hy.moe_route_all(zr, None, experts + 2, top, 1.5, ids=ids, wts=wts))
+        sec = tm(lambda: hy.moe_route_all(zr, None, experts + 2, top, 1.5, ids=ids, wts=wts))
         report(f"{phase}.damilix.moe_route_all", sec, T * ((experts + 2) * 4.0 + top * 8.0))
         z = zr[:, :experts]
-        sec = _time(lambda: hy.moe_route(z, None, top, ids=ids, wts=wts, sigmoid=True))
+        sec = tm(lambda: hy.moe_route(z, None, top, ids=ids, wts=wts, sigmoid=True))
         report(f"{phase}.moe_route(sigmoid)", sec, T * (experts * 4.0 + top * 8.0))
         wg = (torch.randn(experts * 2 * ff, width, device=dev) * width ** -0.5).bfloat16()
         wd = (torch.randn(experts * width, ff, device=dev) * ff ** -0.5).bfloat16()
         res = torch.empty(T, width, **f32)
         wbytes = min(experts, T * top) * 3.0 * ff * width * 2.0
         fl = 6.0 * T * top * width * ff
-        it, wm = (5, 2) if phase == "prefill" else (20, 5)
-        sec = _time(lambda: hy.moe_grouped_ffn(h2, ids, wts, wg, wd, experts, ff, None, fused_act=True, weight_input=True), iters=it, warm=wm)
+        sec = tm(lambda: hy.moe_grouped_ffn(h2, ids, wts, wg, wd, experts, ff, None, fused_act=True, weight_input=True))
         report(f"{phase}.moe_grouped_ffn(weights on the input)", sec, wbytes + T * width * (2.0 + 4.0 * top), flops=fl)
-        sec = _time(lambda: hy.moe_grouped_ffn(h2, ids, wts, wg, wd, experts, ff, res, fused_act=True), iters=it, warm=wm)
+        sec = tm(lambda: hy.moe_grouped_ffn(h2, ids, wts, wg, wd, experts, ff, res, fused_act=True))
         report(f"{phase}.damilix.moe_grouped_ffn(weights on the result)", sec, wbytes + T * width * 6.0, flops=fl)
         del wg, wd
     return out

@@ -1238,8 +1238,8 @@ cudaError_t nrl_parallel_boundary(const float* x_in, const void* embed, int w_f3
       (h1 != nullptr && mu != nullptr && (state == nullptr || carry == nullptr)) || (commit == nullptr) != (commit_state == nullptr) ||
       (x_out != nullptr && x_out == x_in))
     return cudaErrorInvalidValue;
-  // tokens per block: one while that fills the GPU, up to eight (the row above a block is read once more per block)
-  const int rows = T >= 8192 ? 8 : T >= 4096 ? 4 : T >= 2048 ? 2 : 1;
+  // tokens per block: one while that fills the GPU, up to six (the row above a block is read once more per block)
+  const int rows = T >= 8192 ? 6 : T >= 4096 ? 4 : T >= 2048 ? 3 : 1;
   const ParallelBoundary p = {x_in, embed, tok, o, y, slot_of, top, w1, w2, mu, eps, x_out, raw, h1, h2, cu, tok_entry, start, state_slot,
                               state, carry, commit, commit_state, T, W, rows};
   auto ok = [](const void* q, size_t a) { return q == nullptr || aligned(q, a); };
@@ -1247,7 +1247,7 @@ cudaError_t nrl_parallel_boundary(const float* x_in, const void* embed, int w_f3
   const bool vec = W % 4 == 0 && ok(x_in, 16) && ok(o, 16) && ok(y, 16) && ok(w1, 16) && ok(w2, 16) && ok(mu, 16) && ok(x_out, 16) &&
                    ok(state, 16) && ok(carry, 16) && ok(commit, 16) && ok(commit_state, 16) && ok(raw, ha) && ok(h1, ha) && ok(h2, ha);
   const int per = vec ? W / 4 : W;
-  const int th = per <= 64 ? 64 : per <= 128 ? 128 : 256;
+  const int th = per <= 64 ? 64 : per <= 256 ? 128 : 256;
   const int blocks = (T + rows - 1) / rows;
 #define NRL_PB(WT_, HT_, V_)                                                                                             \
   do {                                                                                                                   \

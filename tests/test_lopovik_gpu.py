@@ -158,10 +158,10 @@ class _HostPlan:
         self.tokens = tokens.int().cuda()
 
 
-@pytest.mark.parametrize("W,counts", [(44, [5, 1, 9]), (51, [3, 2]), (1028, [1, 1, 4]), (12, [700, 1, 1360]), (12, [4096, 3]), (20, [1, 8000, 300])])
+@pytest.mark.parametrize("W,counts", [(44, [5, 1, 9]), (51, [3, 2]), (1028, [1, 1, 4]), (516, [3, 1]), (4104, [2, 3]), (4096, [1, 2]), (12, [700, 1, 1360]), (12, [4096, 3]), (20, [1, 8000, 300])])
 def test_boundary_adds_norms_and_shifts(W, counts):
     """Sum of stream, result and gathered expert rows; both norms; the shift inside an entry, at its first token (zeros or the slot's
-    row) and across the rows of different blocks (one to eight tokens per block); what is carried and what is handed over."""
+    row) and across the rows of different blocks (one to six tokens per block); what is carried and what is handed over."""
     from nanorlhf_b200.ops import hybrid as hy
     g = torch.Generator().manual_seed(W)
     E, T, eps, top = len(counts), sum(counts), 1e-5, 2
