@@ -314,7 +314,7 @@ def _pool():
     global _POOL, _POOL_BROKEN
     if _POOL is None and not _POOL_BROKEN:
         ctx = mp.get_context("spawn")
-        _POOL = ctx.Pool(2, maxtasksperchild=500)
+        _POOL = ctx.Pool(2, initializer=_warm, maxtasksperchild=500)      # no worker takes a task before it has imported sympy
         try:                      # pay the interpreter + sympy import once, outside any per-answer timeout
             _POOL.apply_async(_warm).get(60)
         except Exception:
