@@ -196,7 +196,7 @@ __global__ void window_attention_kernel(const float* __restrict__ q, long sq, co
   const int Hv = md.v_div > 1 ? Hkv / md.v_div : Hkv, gv = md.v_div > 1 ? g / md.v_div : g;
   if (md.head_scale != nullptr) scale *= md.head_scale[h];
   const float slope = md.head_slope != nullptr ? md.head_slope[h] : 0.f;
-  if (md.gate != nullptr) out_scale *= sigmoid_(md.gate[t * md.gate_stride + h]);
+  if (md.gate != nullptr && !md.gate_cols) out_scale *= sigmoid_(md.gate[t * md.gate_stride + h]);
   float m = -INFINITY, l = 0.f;
   float acc[kMaxDvPerLane];
 #pragma unroll
@@ -254,7 +254,8 @@ __global__ void window_attention_kernel(const float* __restrict__ q, long sq, co
   for (int c = threadIdx.x; c < Dv; c += blockDim.x) {
     float a = 0.f;
     for (int i = 0; i < kWarps; ++i) a += f[i] * accs[i * Dv + c];
-    const float val = out_scale * (a / lt);
+    float val = out_scale * (a / lt);
+    if (md.gate != nullptr && md.gate_cols) val *= sigmoid_(md.gate[t * md.gate_stride + static_cast<long>(h) * Dv + c]);
     if (md.out_float != nullptr) md.out_float[t * md.out_float_stride + static_cast<long>(h) * Dv + c] = val;
     else st(out, t * so + static_cast<long>(h) * Dv + c, val);
   }
@@ -442,8 +443,8 @@ window_attention_tile_kernel(const float* __restrict__ q, long sq, const CT* __r
         a += f * racc[(static_cast<long>(x) * NQ + qi) * Dv + c];
       }
       float os = out_scale;
-      if (md.gate != nullptr) os *= sigmoid_(md.gate[static_cast<long>(t + qi / hb) * md.gate_stride + h0 + qi % hb]);
       const long orow = t + qi / hb, ocol = static_cast<long>(h0 + qi % hb) * Dv + c;
+      if (md.gate != nullptr) os *= sigmoid_(md.gate[orow * md.gate_stride + (md.gate_cols ? ocol : h0 + qi % hb)]);
       if (md.out_float != nullptr) md.out_float[orow * md.out_float_stride + ocol] = os * (a / lt);
       else st(out, orow * so + ocol, os * (a / lt));
     }
@@ -666,6 +667,7 @@ cudaError_t nrl_window_attention(const float* q, long sq, const void* k_cache, c
   if (md.kv_shared && (Dv > D || v_cache != k_cache)) return cudaErrorInvalidValue;
   if (md.v_div > 1 && (Hkv % md.v_div != 0 || md.kv_shared)) return cudaErrorInvalidValue;
   if (md.dist_bias != nullptr && md.dist_max < 0) return cudaErrorInvalidValue;
+  if (md.gate_cols && md.kv_shared) return cudaErrorInvalidValue;
   // latent attention (one shared row per token is key and value of every head, causal) over bf16 pages: its own tensor-core kernels
   if ((impl == 0 || impl == 3) && !cache_f32 && md.kv_shared && Hkv == 1 && window >= (1 << 30) && !md.chunked &&
       md.head_scale == nullptr && md.head_slope == nullptr && nrl_latent_attention_mma_fits(out, so, D, Dv, page))

@@ -350,18 +350,25 @@ window_attention_mma_kernel(const float* __restrict__ q, long sq, const __nv_bfl
       const float fo = ex2(m_run[hf] - mt);
       f = out_scale * fo / (l * fo + ex2(s2 - mt));
     }
-    if (md.gate != nullptr) f *= sigmoid_(md.gate[static_cast<long>(row_t[hf]) * md.gate_stride + h0 + r % HB]);
+    const float* gcol = nullptr;                           // one gate per output column
+    if (md.gate != nullptr && md.gate_cols) gcol = md.gate + static_cast<long>(row_t[hf]) * md.gate_stride + static_cast<long>(h0 + r % HB) * Dv;
+    else if (md.gate != nullptr) f *= sigmoid_(md.gate[static_cast<long>(row_t[hf]) * md.gate_stride + h0 + r % HB]);
     float* dstf = md.out_float != nullptr
                       ? md.out_float + static_cast<long>(row_t[hf]) * md.out_float_stride + static_cast<long>(h0 + r % HB) * Dv : nullptr;
 #pragma unroll
     for (int i = 0; i < 2 * NV; ++i) {
       const int c = i * 8 + 2 * tq;
       if (c < Dv) {
+        float r0 = o[i][2 * hf] * f, r1 = o[i][2 * hf + 1] * f;
+        if (gcol != nullptr) {
+          r0 *= sigmoid_(gcol[c]);
+          r1 *= sigmoid_(gcol[c + 1]);
+        }
         if (dstf != nullptr) {
-          dstf[c] = o[i][2 * hf] * f;
-          dstf[c + 1] = o[i][2 * hf + 1] * f;
+          dstf[c] = r0;
+          dstf[c + 1] = r1;
         } else {
-          *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(o[i][2 * hf] * f, o[i][2 * hf + 1] * f);
+          *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(r0, r1);
         }
       }
     }
@@ -569,10 +576,10 @@ window_attention_decode_kernel(const float* __restrict__ q, long sq, const __nv_
 // block per (token, query head): out = out_scale * sum_s 2^(m_s - M) O_s / sum_s 2^(m_s - M) l_s
 __global__ void window_attention_merge_kernel(const float* __restrict__ part, int nsplit, int Hq, int Dv, float out_scale,
                                               __nv_bfloat16* __restrict__ out, long so, const float* __restrict__ gate, long gate_stride,
-                                              const float* __restrict__ head_sink, float* __restrict__ out_float, long out_float_stride) {
+                                              int gate_cols, const float* __restrict__ head_sink, float* __restrict__ out_float, long out_float_stride) {
   const long t = blockIdx.x;
   const int h = blockIdx.y;
-  if (gate != nullptr) out_scale *= sigmoid_(gate[t * gate_stride + h]);
+  if (gate != nullptr && !gate_cols) out_scale *= sigmoid_(gate[t * gate_stride + h]);
   const float* p = part + (t * Hq + h) * nsplit * (Dv + 2);
   const float sink2 = head_sink != nullptr ? head_sink[h] * 1.4426950408889634f : -INFINITY;   // the sink joins as a part without values
   float M = sink2;
@@ -588,8 +595,10 @@ __global__ void window_attention_merge_kernel(const float* __restrict__ part, in
       const float m = p[x * (Dv + 2) + Dv];
       if (m != -INFINITY) a += ex2(m - M) * p[x * (Dv + 2) + c];
     }
-    if (out_float != nullptr) out_float[t * out_float_stride + static_cast<long>(h) * Dv + c] = out_scale * (a / L);
-    else out[t * so + static_cast<long>(h) * Dv + c] = __float2bfloat16_rn(out_scale * (a / L));
+    float val = out_scale * (a / L);
+    if (gate != nullptr && gate_cols) val *= sigmoid_(gate[t * gate_stride + static_cast<long>(h) * Dv + c]);
+    if (out_float != nullptr) out_float[t * out_float_stride + static_cast<long>(h) * Dv + c] = val;
+    else out[t * so + static_cast<long>(h) * Dv + c] = __float2bfloat16_rn(val);
   }
 }
 
@@ -636,7 +645,7 @@ cudaError_t launch_decode(const float* q, long sq, const void* k_cache, const vo
   if (e != cudaSuccess) return e;
   window_attention_merge_kernel<<<dim3(T, Hq), Dv <= 32 ? 32 : Dv <= 64 ? 64 : 128, 0, s>>>(part, nsplit * 4, Hq, Dv, out_scale,
                                                                                           static_cast<__nv_bfloat16*>(out), so, md.gate,
-                                                                                          md.gate_stride, md.head_sink, md.out_float, md.out_float_stride);
+                                                                                          md.gate_stride, md.gate_cols, md.head_sink, md.out_float, md.out_float_stride);
   return cudaGetLastError();
 }
 

@@ -5,6 +5,8 @@
 #include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
 
+#include <limits>
+
 #include "gemm_tc.h"
 #include "hybrid_kernels.h"
 #include "tma_host.h"
@@ -208,7 +210,9 @@ void window_attention(const Tensor& q, const Tensor& k_cache, const Tensor& v_ca
     md.head_slope = f32(*head_slope, "head_slope");
   }
   if (gate.has_value()) {
-    TORCH_CHECK(gate->dim() == 2 && gate->size(0) == T && gate->size(1) == Hq, "window_attention: gate [T, Hq]");
+    md.gate_cols = gate->dim() == 2 && gate->size(1) != Hq;
+    TORCH_CHECK(gate->dim() == 2 && gate->size(0) == T && (gate->size(1) == Hq || (!kv_shared && gate->size(1) == static_cast<int64_t>(Hq) * Dv)),
+                "window_attention: gate [T, Hq] or [T, Hq * Dv]");
     md.gate = f32(*gate, "gate");
     md.gate_stride = gate->stride(0);
   }
@@ -490,34 +494,34 @@ void side_gate(const Tensor& u, const Tensor& table, int64_t col0, const Tensor&
         "side_gate");
 }
 
-void swiglu_cols(const Tensor& in, const c10::optional<Tensor>& rgate, Tensor out) {
+void swiglu_cols(const Tensor& in, const c10::optional<Tensor>& rgate, Tensor out, double alpha, double limit, double up_shift) {
   c10::cuda::CUDAGuard guard(in.device());
   TORCH_CHECK(in.dim() == 2 && out.dim() == 2 && in.size(0) == out.size(0) && in.size(1) == 2 * out.size(1), "swiglu_cols: in [T, 2 C], out [T, C]");
   if (rgate.has_value()) TORCH_CHECK(rgate->dim() == 2 && rgate->size(0) == in.size(0) && rgate->size(1) == 1, "swiglu_cols: rgate [T, 1]");
   check(nrl_swiglu_cols(f32(in, "in"), in.stride(0), rgate.has_value() ? f32(*rgate, "rgate") : nullptr,
-                        rgate.has_value() ? rgate->stride(0) : 0, out.data_ptr(), out.stride(0), typed(out, "out"),
-                        static_cast<int>(in.size(0)), static_cast<int>(out.size(1)), cur_stream()),
+                        rgate.has_value() ? rgate->stride(0) : 0, static_cast<float>(alpha), static_cast<float>(limit), static_cast<float>(up_shift),
+                        out.data_ptr(), out.stride(0), typed(out, "out"), static_cast<int>(in.size(0)), static_cast<int>(out.size(1)), cur_stream()),
         "swiglu_cols");
 }
 
 void moe_route_all(const Tensor& router, const c10::optional<Tensor>& correction, int64_t n_real, int64_t top, double route_scale,
                    int64_t groups, int64_t keep, const c10::optional<Tensor>& gu, int64_t ff, const c10::optional<Tensor>& act, const c10::optional<Tensor>& ids,
-                   const c10::optional<Tensor>& wts, const c10::optional<Tensor>& self_w) {
+                   const c10::optional<Tensor>& wts, const c10::optional<Tensor>& self_w, bool sigmoid, bool group_sum2, bool relu2) {
   c10::cuda::CUDAGuard guard(router.device());
   TORCH_CHECK(router.dim() == 2, "moe_route_all: router [T, E]");
   const int T = static_cast<int>(router.size(0)), E = static_cast<int>(router.size(1));
   if (correction.has_value()) TORCH_CHECK(correction->numel() == E, "moe_route_all: correction [E]");
   TORCH_CHECK(act.has_value() == gu.has_value(), "moe_route_all: gu and act go together");
   if (act.has_value())
-    TORCH_CHECK(gu->dim() == 2 && gu->size(0) == T && gu->size(1) == n_real * 2 * ff && act->dim() == 2 && act->size(0) == T &&
-                    act->size(1) == n_real * ff, "moe_route_all: gu [T, n_real*2ff], act [T, n_real*ff]");
+    TORCH_CHECK(gu->dim() == 2 && gu->size(0) == T && gu->size(1) == n_real * (relu2 ? 1 : 2) * ff && act->dim() == 2 && act->size(0) == T &&
+                    act->size(1) == n_real * ff, "moe_route_all: gu [T, n_real*2ff] (relu2: [T, n_real*ff]), act [T, n_real*ff]");
   if (ids.has_value()) TORCH_CHECK(ids->scalar_type() == torch::kInt32 && ids->is_contiguous() && ids->numel() == static_cast<int64_t>(T) * top, "moe_route_all: ids int32 [T, top]");
   if (wts.has_value()) TORCH_CHECK(wts->is_contiguous() && wts->numel() == static_cast<int64_t>(T) * top, "moe_route_all: wts float [T, top]");
   if (self_w.has_value()) TORCH_CHECK(self_w->is_contiguous() && self_w->numel() == T, "moe_route_all: self_w float [T]");
   Tensor wt = wts.has_value() ? *wts : Tensor(), sw = self_w.has_value() ? *self_w : Tensor();
   check(nrl_moe_route_all(f32(router, "router"), router.stride(0), correction.has_value() ? f32(*correction, "correction") : nullptr, E,
-                          static_cast<int>(n_real), static_cast<int>(top), static_cast<float>(route_scale), static_cast<int>(groups),
-                          static_cast<int>(keep), gu.has_value() ? f32(*gu, "gu") : nullptr, gu.has_value() ? gu->stride(0) : 0, static_cast<int>(ff),
+                          static_cast<int>(n_real), static_cast<int>(top), static_cast<float>(route_scale), sigmoid ? 1 : 0, static_cast<int>(groups),
+                          static_cast<int>(keep), group_sum2 ? 1 : 0, relu2 ? 1 : 0, gu.has_value() ? f32(*gu, "gu") : nullptr, gu.has_value() ? gu->stride(0) : 0, static_cast<int>(ff),
                           act.has_value() ? act->data_ptr() : nullptr, act.has_value() ? act->stride(0) : 0,
                           act.has_value() ? typed(*act, "act") : 1, ids.has_value() ? ids->data_ptr<int>() : nullptr,
                           wts.has_value() ? f32w(wt, "wts") : nullptr, self_w.has_value() ? f32w(sw, "self_w") : nullptr, T, cur_stream()),
@@ -568,7 +572,7 @@ void parallel_boundary(const c10::optional<Tensor>& x_in, const Tensor& embed, c
                        const c10::optional<Tensor>& w2, const c10::optional<Tensor>& mu, double eps, c10::optional<Tensor> x_out,
                        c10::optional<Tensor> raw, c10::optional<Tensor> h1, c10::optional<Tensor> h2, const Tensor& cu, const Tensor& tok_entry,
                        const Tensor& start, const Tensor& state_slot, const c10::optional<Tensor>& state, c10::optional<Tensor> carry,
-                       const c10::optional<Tensor>& commit, c10::optional<Tensor> commit_state) {
+                       const c10::optional<Tensor>& commit, c10::optional<Tensor> commit_state, const c10::optional<Tensor>& wts) {
   c10::cuda::CUDAGuard guard(embed.device());
   const int T = static_cast<int>(tok.numel()), W = static_cast<int>(embed.size(1)), E = static_cast<int>(start.numel());
   TORCH_CHECK(embed.dim() == 2 && embed.is_contiguous(), "parallel_boundary: embed [V, W]");
@@ -601,15 +605,35 @@ void parallel_boundary(const c10::optional<Tensor>& x_in, const Tensor& embed, c
     TORCH_CHECK(T > 0 && slot_of->numel() % T == 0 && slot_of->numel() == y->size(0), "parallel_boundary: slot_of [T, top] names the rows of y");
     top = static_cast<int>(slot_of->numel() / T);
   }
+  if (wts.has_value()) TORCH_CHECK(y.has_value() && wts->is_contiguous() && wts->numel() == slot_of->numel(), "parallel_boundary: wts [T, top] goes with y");
   const float* cs = rows(commit_state, "commit_state", -1);
   const float* st = rows(state, "state", -1);
   check(nrl_parallel_boundary(rows(x_in, "x_in", T), x_in.has_value() ? nullptr : embed.data_ptr(), typed(embed, "embed"), i32(tok, "tok"),
-                              rows(o, "o", T), rows(y, "y", -1), slot_of.has_value() ? i32(*slot_of, "slot_of") : nullptr, top, vec(w1, "w1"),
+                              rows(o, "o", T), rows(y, "y", -1), slot_of.has_value() ? i32(*slot_of, "slot_of") : nullptr, wts.has_value() ? f32(*wts, "wts") : nullptr, top, vec(w1, "w1"),
                               vec(w2, "w2"), vec(mu, "mu"), static_cast<float>(eps), const_cast<float*>(rows(x_out, "x_out", T)), rp, p1, p2,
                               h_f32 == 1 ? 1 : 0, i32(cu, "cu"), i32(tok_entry, "tok_entry"), i32(start, "start"),
                               i32(state_slot, "state_slot"), st, const_cast<float*>(rows(carry, "carry", E)), rows(commit, "commit", E),
                               const_cast<float*>(cs), T, W, cur_stream()),
         "parallel_boundary");
+}
+
+// ---- linear attention with a constant decay per head ----
+void lightning_scan(const Tensor& qkv, int64_t col_q, int64_t col_k, int64_t col_v, const Tensor& pows, Tensor state, Tensor o, const Tensor& cu,
+                    const Tensor& start, const Tensor& state_slot, bool chunk_ok, int64_t impl) {
+  c10::cuda::CUDAGuard guard(o.device());
+  TORCH_CHECK(state.dim() == 4 && state.is_contiguous(), "lightning_scan: state [slots, heads, D, Dv]");
+  const int heads = static_cast<int>(state.size(1)), D = static_cast<int>(state.size(2)), Dv = static_cast<int>(state.size(3));
+  const int E = static_cast<int>(start.numel());
+  TORCH_CHECK(qkv.dim() == 2 && col_q >= 0 && col_k >= 0 && col_v >= 0 && col_q + heads * D <= qkv.size(1) && col_k + heads * D <= qkv.size(1) &&
+                  col_v + heads * Dv <= qkv.size(1) && o.is_contiguous() && o.dim() == 2 && o.size(0) == qkv.size(0) && o.size(1) == heads * Dv,
+              "lightning_scan: shapes");
+  TORCH_CHECK(pows.dim() == 2 && pows.size(0) == heads && pows.size(1) >= 2 && pows.is_contiguous(), "lightning_scan: pows [heads, powers]");
+  TORCH_CHECK(cu.numel() == E + 1 && state_slot.numel() == E, "lightning_scan: plan");
+  check(nrl_lightning_scan(f32(qkv, "qkv"), qkv.stride(0), static_cast<int>(col_q), static_cast<int>(col_k), static_cast<int>(col_v),
+                           f32(pows, "pows"), static_cast<int>(pows.size(1)), f32w(state, "state"), f32w(o, "o"), i32(cu, "cu"), i32(start, "start"),
+                           i32(state_slot, "state_slot"), E, heads, D, Dv, qkv.size(0) == E ? 1 : 0, chunk_ok ? 1 : 0, static_cast<int>(impl),
+                           cur_stream()),
+        "lightning_scan");
 }
 
 void gate_cols(const Tensor& in, const Tensor& gate, double scale, Tensor out) {
@@ -674,14 +698,14 @@ void moe_combine(const Tensor& y, const Tensor& slot_of, const Tensor& wts, Tens
 //   out float [R, N] = a[r] . b[expert(r)]^T,  or
 //   (row_scale float [R] then multiplies gate and up first)  act bf16 [R, N / 2] = silu(gate) * up with b's rows interleaved per 32 features ([32 gate rows | 32 up rows], N % 64 == 0).
 void gemm_tc_grouped(const Tensor& a, const Tensor& b, const c10::optional<Tensor>& out, const Tensor& tiles, const Tensor& num_tiles,
-                     int64_t block_n, const c10::optional<Tensor>& act, const c10::optional<Tensor>& row_scale) {
+                     int64_t block_n, const c10::optional<Tensor>& act, const c10::optional<Tensor>& row_scale, bool relu2) {
   c10::cuda::CUDAGuard guard(a.device());
   TORCH_CHECK(a.is_cuda() && b.is_cuda() && a.scalar_type() == torch::kBFloat16 && b.scalar_type() == torch::kBFloat16 && a.dim() == 2 &&
                   b.dim() == 2 && a.stride(1) == 1 && b.stride(1) == 1, "gemm_tc_grouped: bf16 2D operands with unit inner stride");
   TORCH_CHECK((a.stride(0) * 2) % 16 == 0 && (b.stride(0) * 2) % 16 == 0 && (reinterpret_cast<uintptr_t>(a.data_ptr()) & 15) == 0 &&
                   (reinterpret_cast<uintptr_t>(b.data_ptr()) & 15) == 0, "gemm_tc_grouped: 16-byte aligned rows");
   TORCH_CHECK(out.has_value() != act.has_value(), "gemm_tc_grouped: give either the float result or the activation output");
-  const int64_t R = a.size(0), K = a.size(1), N = out.has_value() ? out->size(1) : 2 * act->size(1);
+  const int64_t R = a.size(0), K = a.size(1), N = out.has_value() ? out->size(1) : (relu2 ? 1 : 2) * act->size(1);
   TORCH_CHECK(b.size(1) == K && K % 8 == 0 && N % 8 == 0 && b.size(0) % N == 0, "gemm_tc_grouped: b [E * N, K], K and N multiples of 8");
   TORCH_CHECK(tiles.scalar_type() == torch::kInt32 && tiles.is_contiguous() && tiles.dim() == 2 && tiles.size(1) == 3 &&
                   num_tiles.scalar_type() == torch::kInt32 && num_tiles.numel() == 1, "gemm_tc_grouped: tile table");
@@ -694,8 +718,9 @@ void gemm_tc_grouped(const Tensor& a, const Tensor& b, const c10::optional<Tenso
     p.out_f32_stride = out->stride(0);
   } else {
     TORCH_CHECK(act->scalar_type() == torch::kBFloat16 && act->dim() == 2 && act->size(0) == R && act->stride(1) == 1 &&
-                    act->stride(0) % 8 == 0 && (reinterpret_cast<uintptr_t>(act->data_ptr()) & 15) == 0 && N % 64 == 0,
-                "gemm_tc_grouped: act bf16 [R, N / 2], 16-byte aligned rows, N a multiple of 64");
+                    act->stride(0) % 8 == 0 && (reinterpret_cast<uintptr_t>(act->data_ptr()) & 15) == 0 && (relu2 || N % 64 == 0),
+                "gemm_tc_grouped: act bf16 [R, N / 2], 16-byte aligned rows, N a multiple of 64 (relu2: act [R, N])");
+    p.act = relu2 ? 2 : 0;
     p.out_bf16 = reinterpret_cast<__nv_bfloat16*>(act->data_ptr());
     p.out_stride = act->stride(0);
   }
@@ -732,12 +757,19 @@ void bind_hybrid(pybind11::module_& m) {
   m.def("moe_combine", &moe_combine, "out[t] = sum_k wts[t, k] y[slot_of[t, k]]");
   m.def("gemm_tc_grouped", &gemm_tc_grouped, "grouped tcgen05 GEMM over rows sorted by expert: float32 out, or fused SwiGLU bf16 out",
         pybind11::arg("a"), pybind11::arg("b"), pybind11::arg("out"), pybind11::arg("tiles"), pybind11::arg("num_tiles"),
-        pybind11::arg("block_n") = 0, pybind11::arg("act") = pybind11::none(), pybind11::arg("row_scale") = pybind11::none());
+        pybind11::arg("block_n") = 0, pybind11::arg("act") = pybind11::none(), pybind11::arg("row_scale") = pybind11::none(),
+        pybind11::arg("relu2") = false);
   m.def("embed_norm", &embed_norm, "x = rmsnorm(embed[tok]) * w (float), h = x (typed)");
   m.def("post_norm_residual", &post_norm_residual, "x += rmsnorm(o + self_w x) * w_post; h = w_pre ? rmsnorm(x) * w_pre : x");
   m.def("side_gate", &side_gate, "out = gelu_tanh(u) * table[tok, col0:col0 + C], zero padded");
-  m.def("swiglu_cols", &swiglu_cols, "out = silu(in[:, :C]) * in[:, C:] * sigmoid(row gate)");
-  m.def("moe_route_all", &moe_route_all, "routing by a softmax over all router outputs, with identity experts");
+  m.def("swiglu_cols", &swiglu_cols, "out = g sigmoid(alpha g) * (u + up_shift) * sigmoid(row gate), g = in[:, :C], u = in[:, C:], both clamped",
+        pybind11::arg("in"), pybind11::arg("rgate"), pybind11::arg("out"), pybind11::arg("alpha") = 1.0,
+        pybind11::arg("limit") = std::numeric_limits<double>::infinity(), pybind11::arg("up_shift") = 0.0);
+  m.def("moe_route_all", &moe_route_all, "routing by a softmax or sigmoids over all router outputs, with groups and identity experts",
+        pybind11::arg("router"), pybind11::arg("correction"), pybind11::arg("n_real"), pybind11::arg("top"), pybind11::arg("route_scale"),
+        pybind11::arg("groups"), pybind11::arg("keep"), pybind11::arg("gu"), pybind11::arg("ff"), pybind11::arg("act"), pybind11::arg("ids"),
+        pybind11::arg("wts"), pybind11::arg("self_w"), pybind11::arg("sigmoid") = false, pybind11::arg("group_sum2") = false,
+        pybind11::arg("relu2") = false);
   m.def("gla_prep", &gla_prep, "q * D^-1/2 in place and per-channel decays sigmoid(z)^(1/tau) of gated linear attention");
   m.def("latent_kv_write", &latent_kv_write, "normed latent + rotated shared key part into the page; rotated query parts into the absorbed queries");
   m.def("embed_pos", &embed_pos, "x0 = embed[tok] + pos_table[pos] (float)");
@@ -772,7 +804,13 @@ void bind_hybrid(pybind11::module_& m) {
         pybind11::arg("router"), pybind11::arg("router_bias"), pybind11::arg("top"), pybind11::arg("gu"), pybind11::arg("ff"),
         pybind11::arg("act"), pybind11::arg("ids"), pybind11::arg("wts"), pybind11::arg("sigmoid") = false,
         pybind11::arg("weight_input") = false);
-  m.def("parallel_boundary", &parallel_boundary, "x += results; two RMS norms of x, the first with a token shift carried per slot");
+  m.def("parallel_boundary", &parallel_boundary, "x += results; two RMS norms of x, the first with a token shift carried per slot", pybind11::arg("x_in"),
+        pybind11::arg("embed"), pybind11::arg("tok"), pybind11::arg("o"), pybind11::arg("y"), pybind11::arg("slot_of"), pybind11::arg("w1"),
+        pybind11::arg("w2"), pybind11::arg("mu"), pybind11::arg("eps"), pybind11::arg("x_out"), pybind11::arg("raw"), pybind11::arg("h1"),
+        pybind11::arg("h2"), pybind11::arg("cu"), pybind11::arg("tok_entry"), pybind11::arg("start"), pybind11::arg("state_slot"),
+        pybind11::arg("state"), pybind11::arg("carry"), pybind11::arg("commit"), pybind11::arg("commit_state"),
+        pybind11::arg("wts") = pybind11::none());
+  m.def("lightning_scan", &lightning_scan, "linear attention with a constant decay per head over silu'd projections, state carried per slot");
   m.def("gate_cols", &gate_cols, "out = scale * in * sigmoid(gate)");
 }
 }  // namespace nrl

@@ -443,7 +443,26 @@ NRL_DEVICE void gemm_tc_body(const CUtensorMap& tmA, const CUtensorMap& tmB, con
           }
         }
         const int col0 = c.n_blk * BN + ch * 64;
-        if (EPI == EPI_F32 && GROUPED && p.out_bf16 != nullptr) {
+        if (EPI == EPI_F32 && GROUPED && p.out_bf16 != nullptr && p.act == 2) {
+          // grouped up projection with the squared ReLU formed here: a chunk yields 64 activations of this row
+          if (row_ok) {
+            const float rw = p.row_scale != nullptr ? p.row_scale[row] : 1.f;
+            __nv_bfloat16* orow = p.out_bf16 + static_cast<long>(row) * p.out_stride + col0;
+#pragma unroll
+            for (int h = 0; h < 2; ++h)
+#pragma unroll
+              for (int j = 0; j < 32; j += 8) {
+                if (col0 + h * 32 + j >= p.N) continue;     // N % 8 == 0
+                uint32_t pk[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  const float a0 = fmaxf(rw * __uint_as_float(v[h][j + 2 * e]), 0.f), a1 = fmaxf(rw * __uint_as_float(v[h][j + 2 * e + 1]), 0.f);
+                  pk[e] = pack_bf16x2(a0 * a0, a1 * a1);
+                }
+                *reinterpret_cast<uint4*>(orow + h * 32 + j) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+              }
+          }
+        } else if (EPI == EPI_F32 && GROUPED && p.out_bf16 != nullptr) {
           // grouped gate / up projection with the SwiGLU formed here: B rows are interleaved per 32 features ([32 gate | 32 up]
           // in every 64-column chunk), so a chunk yields 32 activations of this row: 64 contiguous bytes, plain masked stores
           const int f0 = c.n_blk * (BN / 2) + ch * 32;
@@ -779,7 +798,7 @@ extern "C" cudaError_t nrl_gemm_tc_grouped(const CUtensorMap* maps, const nrl::t
                                            cudaStream_t stream) {
   using namespace nrl::tc;
   if (p->grp_tiles == nullptr || p->grp_num_tiles == nullptr || p->K2 != 0 || max_tiles < 1 || p->N % 4 != 0) return cudaErrorInvalidValue;
-  if (p->out_bf16 == nullptr ? p->out_f32 == nullptr : (p->N % 64 != 0 || p->out_stride % 8 != 0)) return cudaErrorInvalidValue;
+  if (p->out_bf16 == nullptr ? p->out_f32 == nullptr : (p->N % (p->act == 2 ? 8 : 64) != 0 || p->out_stride % 8 != 0)) return cudaErrorInvalidValue;
   if (bn == 64) return launch_grouped<64>(maps, *p, max_tiles, num_sms, stream);
   if (bn == 128) return launch_grouped<128>(maps, *p, max_tiles, num_sms, stream);
   if (bn == 256) return launch_grouped<256>(maps, *p, max_tiles, num_sms, stream);

@@ -21,7 +21,7 @@ struct TcParams {
   int batch;                    // BATCH kernels: number of independent [M,K] x [N,K]^T problems behind 3D tensor maps (else 1)
   float alpha;                  // multiplies the accumulator
   const __nv_bfloat16* bias;    // EPI_BF16: optional [N]
-  int act;                      // EPI_BF16: 0 = none, 1 = exact (erf) GELU after the bias
+  int act;                      // EPI_BF16: 0 = none, 1 = exact (erf) GELU after the bias (GROUPED: see below)
   float* out_f32;               // EPI_F32: [M, N] fp32, row stride out_f32_stride elements
   long out_f32_stride;
   int accumulate;               // EPI_F32: 1 = add to what is there
@@ -54,7 +54,8 @@ extern "C" cudaError_t nrl_gemm_tc_batched(const CUtensorMap* maps, const nrl::t
 // grouped K-major x K-major GEMM (cta_group 1); maps = {A [rows, K] box {128, 64}, B [experts * N, K] box {bn, 64}};
 // p->N = columns per expert; max_tiles bounds the table's length (grid size).  Output: out_f32 [rows, N], or, when out_bf16 is
 // set, the SwiGLU of the columns: B rows interleaved per 32 features ([32 gate | 32 up], N % 64 == 0), out_bf16 [rows, N / 2]
-// (row stride out_stride, a multiple of 8) = silu(gate) * up; row_scale [rows] (or null) then multiplies gate and up first.
+// (row stride out_stride, a multiple of 8) = silu(gate) * up; row_scale [rows] (or null) then multiplies gate and up first.  act == 2: the
+// squared ReLU of the columns instead, out_bf16 [rows, N] = relu(row_scale * x)^2, B rows in their own order.
 extern "C" cudaError_t nrl_gemm_tc_grouped(const CUtensorMap* maps, const nrl::tc::TcParams* p, int bn, int max_tiles, int num_sms,
                                            cudaStream_t stream);
 extern "C" cudaError_t nrl_gemm_tc(const CUtensorMap* maps, const nrl::tc::TcParams* p, int cg, int bn, int a_mn, int b_mn,

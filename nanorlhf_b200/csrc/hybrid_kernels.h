@@ -32,6 +32,7 @@ typedef struct {
                              // score maps over one set of values)
   float* out_float;          // non-null: the result goes here as float ([T, Hq * Dv], row stride out_float_stride) whatever the pages'
   long out_float_stride;     // type, and `out` is not written (results that are combined further before they are rounded)
+  int gate_cols;             // 1: `gate` is [T, Hq * Dv], one value per output column instead of one per head (not with kv_shared)
 } NrlAttnMods;
 
 extern "C" {
@@ -90,17 +91,19 @@ cudaError_t nrl_post_norm_residual(float* x, const float* o, const float* self_w
 // (u float, row stride su; table typed, row stride st_).
 cudaError_t nrl_side_gate(const float* u, long su, const void* table, long st_, int w_f32, int col0, const int* tok, void* out, long so,
                           int out_f32, int T, int C, int Cpad, cudaStream_t s);
-// out[t, c] (typed) = silu(in[t, c]) * in[t, C + c] * (rgate ? sigmoid(rgate[t * srg]) : 1)
-cudaError_t nrl_swiglu_cols(const float* in, long si, const float* rgate, long srg, void* out, long so, int out_f32, int T, int C,
-                            cudaStream_t s);
-// Routing by a softmax over all E router outputs; the last E - n_real are identity experts.  The `top` largest
-// softmax + correction (correction [E] or null; ties: lowest index) are chosen; weight = softmax / (sum over the chosen + 1e-20)
+// out[t, c] (typed) = g sigmoid(alpha g) * (u + up_shift) * (rgate ? sigmoid(rgate[t * srg]) : 1), g = in[t, c], u = in[t, C + c];
+// a finite limit caps g from above and u on both sides first.  SwiGLU: alpha 1, limit INFINITY, up_shift 0
+cudaError_t nrl_swiglu_cols(const float* in, long si, const float* rgate, long srg, float alpha, float limit, float up_shift, void* out, long so,
+                            int out_f32, int T, int C, cudaStream_t s);
+// Routing by a score over all E router outputs (sigmoid 0: softmax, 1: each output's own sigmoid); the last E - n_real are identity
+// experts.  The `top` largest score + correction (correction [E] or null; ties: lowest index) are chosen; weight = score / (sum over the chosen + 1e-20)
 // * route_scale.  ids [T, top]; wts [T, top] (0 for a chosen identity expert); self_w [T] = summed weights of the chosen
 // identity experts (needed when n_real < E).  Dense form as nrl_moe_route, over the n_real experts.
+// relu2 1: the dense form's experts are relu(up)^2 (gu holds ff columns per expert) instead of SwiGLU.
 // groups > 1: the E outputs form `groups` equal groups of neighbours; a group's score is its largest choice score (score +
-// correction) and only experts of the `keep` best groups can be chosen (the others count as -inf; ties: the lower group).
+// correction), or with group_sum2 the sum of its two largest, and only experts of the `keep` best groups can be chosen (the others count as -inf; ties: the lower group).
 cudaError_t nrl_moe_route_all(const float* router, long sr, const float* correction, int E, int n_real, int top, float route_scale,
-                              int groups, int keep, const float* gu, long sgu, int ff, void* act, long sa, int act_f32, int* ids,
+                              int sigmoid, int groups, int keep, int group_sum2, int relu2, const float* gu, long sgu, int ff, void* act, long sa, int act_f32, int* ids,
                               float* wts, float* self_w, int T, cudaStream_t s);
 
 // Layer boundary of a depth-weighted residual stream.  results: float [n_results_cap, stride_r] with rows of W.
@@ -221,15 +224,16 @@ cudaError_t nrl_window_attention_mma(const float* q, long sq, const void* k_cach
                                      void* out, long so, int T, int Hq, int Hkv, int D, int Dv, int page, int single_token,
                                      const NrlAttnMods* mods, cudaStream_t s);
 // Boundary of a stream whose mixer and feed-forward read the same x side by side, each behind its own RMS norm (weights per column).
-//   x = (x_in [T, W], or embed[tok] when x_in is null) + o [T, W] + sum_k y[slot_of[t * top + k]]      (o, y may be null)
+//   x = (x_in [T, W], or embed[tok] when x_in is null) + o [T, W] + sum_k wts[t * top + k] y[slot_of[t * top + k]]  (o, y may be null;
+//   wts null: every weight is 1)
 //   x_out (float, not x_in) = x;  raw (typed) = x;  h1 (typed) = x / rms(x) * w1;  h2 (typed) = x / rms(x) * w2      (any may be null)
 //   mu [W] (or null), token shift: h1 <- h1 + (h1 of the sequence's previous token - h1) * mu;  the previous token's h1 of an entry's
 //   first token is its slot's row of state [slots, W] (zeros at position 0);  the last token's h1 goes to carry [entries, W]
 //   commit [entries, W] -> commit_state [slots, W]: hands an EARLIER boundary's carry to its state (one launch never writes the
 //   state it reads)
 cudaError_t nrl_parallel_boundary(const float* x_in, const void* embed, int w_f32, const int* tok, const float* o, const float* y,
-                                  const int* slot_of, int top, const float* w1, const float* w2, const float* mu, float eps, float* x_out,
-                                  void* raw, void* h1, void* h2, int h_f32, const int* cu, const int* tok_entry, const int* start,
+                                  const int* slot_of, const float* wts, int top, const float* w1, const float* w2, const float* mu, float eps,
+                                  float* x_out, void* raw, void* h1, void* h2, int h_f32, const int* cu, const int* tok_entry, const int* start,
                                   const int* state_slot, const float* state, float* carry, const float* commit, float* commit_state, int T,
                                   int W, cudaStream_t s);
 // out[t, c] (typed, row stride so) = scale * in[t, c] * sigmoid(gate[t, c])  (floats, row strides si / sg)
@@ -246,6 +250,20 @@ cudaError_t nrl_embed_streams(const void* embed, int w_f32, const int* tok, floa
 cudaError_t nrl_hyper_boundary(float* xs, int S, const float* o, const float* o_bias, const float* self_w, const float* mix,
                                const float* outw, const float* inw, const float* ln_w, const float* ln_b, float eps, void* h, int h_f32,
                                int T, int W, cudaStream_t s);
+
+// Linear attention with a constant decay per head ("lightning").  qkv float [T, *] (row stride sq): raw projections, q at col_q, k at col_k
+// (heads * D each), v at col_v (heads * Dv); silu is applied to all three here.  Per head  S = d_h S + k v^T;  o = S^T q.
+// pows float [heads, npow]: pows[h, n] = d_h^n (n = 0 .. npow - 1).  state float [slots, heads, D, Dv];  o float [T, heads * Dv].
+// `impl`: 0 picks, 1 token by token with the state in registers, 2 token by token with the state in global memory, 3 chunks of
+// NRL_LIGHTNING_CHUNK tokens on the tensor cores (bf16 operands, float state; D and Dv multiples of 8 up to 128, npow > the chunk).
+// chunk_ok 0: never choose 3.  single_token: every entry holds one token.
+#define NRL_LIGHTNING_CHUNK 64
+cudaError_t nrl_lightning_scan(const float* qkv, long sq, int col_q, int col_k, int col_v, const float* pows, int npow, float* state, float* o,
+                               const int* cu, const int* start, const int* state_slot, int E, int heads, int D, int Dv, int single_token,
+                               int chunk_ok, int impl, cudaStream_t s);
+int nrl_lightning_chunk_fits(int D, int Dv, int npow);
+cudaError_t nrl_lightning_chunk(const float* qkv, long sq, int col_q, int col_k, int col_v, const float* pows, int npow, float* state, float* o,
+                                const int* cu, const int* start, const int* state_slot, int E, int heads, int D, int Dv, cudaStream_t s);
 
 // Matrix memory with exponential gates (mLSTM).  qkv float [T, *] (row stride sq): q at col_q, k at col_k (heads * D each), v at
 // col_v (heads * Dv), raw gates at col_i / col_f (heads each; i_bias / f_bias [heads] or null are added).

@@ -434,17 +434,29 @@ __global__ void side_gate_kernel(const float* __restrict__ u, long su, const WT*
   }
 }
 
-// out[t, c] (typed) = silu(in[t, c]) * in[t, C + c] * (rgate ? sigmoid(rgate[t * srg]) : 1):  SwiGLU over [gate | up] columns with an
-// optional sigmoid gate per row
+// Gated linear unit g * sigmoid(alpha g) * (u + up_shift); a finite limit caps g from above and u on both sides first
+struct GluForm {
+  float alpha, limit, up_shift;
+};
+__device__ __forceinline__ float glu_(float g, float u, const GluForm& f) {
+  if (f.limit < INFINITY) {
+    g = fminf(g, f.limit);
+    u = fminf(fmaxf(u, -f.limit), f.limit);
+  }
+  return g * sigmoidf_(f.alpha * g) * (u + f.up_shift);
+}
+
+// out[t, c] (typed) = glu(in[t, c], in[t, C + c]) * (rgate ? sigmoid(rgate[t * srg]) : 1) over [gate | up] columns with an optional sigmoid
+// gate per row
 template <typename OT>
-__global__ void swiglu_cols_kernel(const float* __restrict__ in, long si, const float* __restrict__ rgate, long srg, OT* __restrict__ out,
-                                   long so, long T, int C) {
+__global__ void swiglu_cols_kernel(const float* __restrict__ in, long si, const float* __restrict__ rgate, long srg, GluForm form,
+                                   OT* __restrict__ out, long so, long T, int C) {
   const long n = T * C;
   for (long idx = blockIdx.x * static_cast<long>(blockDim.x) + threadIdx.x; idx < n; idx += static_cast<long>(gridDim.x) * blockDim.x) {
     const long t = idx / C;
     const int c = static_cast<int>(idx - t * C);
     const float g = in[t * si + c], up = in[t * si + C + c];
-    float v = g * sigmoidf_(g) * up;
+    float v = glu_(g, up, form);
     if (rgate != nullptr) v *= sigmoidf_(rgate[t * srg]);
     st(out, t * so + c, v);
   }
@@ -452,7 +464,7 @@ __global__ void swiglu_cols_kernel(const float* __restrict__ in, long si, const 
 
 // the same, four columns per thread (128-bit loads, 64- / 128-bit stores)
 template <typename OT>
-__global__ void swiglu_cols_vec4_kernel(const float* __restrict__ in, long si, const float* __restrict__ rgate, long srg,
+__global__ void swiglu_cols_vec4_kernel(const float* __restrict__ in, long si, const float* __restrict__ rgate, long srg, GluForm form,
                                         OT* __restrict__ out, long so, long T, int C4) {
   const long n = T * C4;
   for (long idx = blockIdx.x * static_cast<long>(blockDim.x) + threadIdx.x; idx < n; idx += static_cast<long>(gridDim.x) * blockDim.x) {
@@ -463,40 +475,47 @@ __global__ void swiglu_cols_vec4_kernel(const float* __restrict__ in, long si, c
     ldv<4>(in + t * si + 4 * C4 + c, up);
     const float rg = rgate != nullptr ? sigmoidf_(rgate[t * srg]) : 1.f;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) v[i] = g[i] * sigmoidf_(g[i]) * up[i] * rg;
+    for (int i = 0; i < 4; ++i) v[i] = glu_(g[i], up[i], form) * rg;
     st4(out + t * so + c, v);
   }
 }
 
-// Routing by a softmax over ALL router outputs, one warp per token.  E outputs, of which the last E - n_real are identity
-// experts (their result is the expert's input).  s = softmax(z);  the `top` largest s + correction are chosen (ties: lowest
+// Routing by a score over ALL router outputs, one warp per token.  E outputs, of which the last E - n_real are identity
+// experts (their result is the expert's input).  s = softmax(z), or (sigmoid) each output's own sigmoid;  the `top` largest s + correction are chosen (ties: lowest
 // index);  weight = s / (sum of the chosen s + 1e-20) * route_scale.
 //   ids [T, top] int;  wts [T, top] float: the weight, 0 for a chosen identity expert;  self_w [T]: the identity experts' weights, summed
-//   act != nullptr (dense form):  act[t, e*ff + c] = weight_e * silu(gu[t, e*2ff + c]) * gu[t, e*2ff + ff + c] for e < n_real, 0 if not chosen
+//   act != nullptr (dense form):  act[t, e*ff + c] = weight_e * silu(gu[t, e*2ff + c]) * gu[t, e*2ff + ff + c] for e < n_real, 0 if not chosen;
+//     relu2:  weight_e * relu(gu[t, e*ff + c])^2
+// groups: see the header; group_sum2: a group's score is the sum of its two largest choice scores instead of the largest
 template <typename OT>
 __global__ void moe_route_all_kernel(const float* __restrict__ router, long sr, const float* __restrict__ correction, int E, int n_real,
-                                     int top, float route_scale, int groups, int keep, const float* __restrict__ gu, long sgu, int ff,
-                                     OT* __restrict__ act, long sa, int* __restrict__ ids, float* __restrict__ wts,
+                                     int top, float route_scale, int sigmoid, int groups, int keep, int group_sum2, int relu2,
+                                     const float* __restrict__ gu, long sgu, int ff, OT* __restrict__ act, long sa, int* __restrict__ ids, float* __restrict__ wts,
                                      float* __restrict__ self_w) {
   extern __shared__ float smf[];
-  float* sc = smf;                // [E] softmax scores
+  float* sc = smf;                // [E] scores
   float* ch = sc + E;             // [E] choice scores, -inf once taken
   float* wsel = ch + E;           // [E] weight, 0 = not chosen
   __shared__ int chosen[64];
   const long t = blockIdx.x;
   if (threadIdx.x < 32) {
     const int lane = threadIdx.x;
-    float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, router[t * sr + e]);
+    float den = 1.f;
+    if (sigmoid) {
+      for (int e = lane; e < E; e += 32) sc[e] = sigmoidf_(router[t * sr + e]);
+    } else {
+      float mx = -INFINITY;
+      for (int e = lane; e < E; e += 32) mx = fmaxf(mx, router[t * sr + e]);
 #pragma unroll
-    for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-    float den = 0.f;
-    for (int e = lane; e < E; e += 32) {
-      const float p = expf(router[t * sr + e] - mx);
-      sc[e] = p;
-      den += p;
+      for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      den = 0.f;
+      for (int e = lane; e < E; e += 32) {
+        const float p = expf(router[t * sr + e] - mx);
+        sc[e] = p;
+        den += p;
+      }
+      den = warp_sum(den);
     }
-    den = warp_sum(den);
     for (int e = lane; e < E; e += 32) {
       const float p = sc[e] / den;
       sc[e] = p;
@@ -505,12 +524,17 @@ __global__ void moe_route_all_kernel(const float* __restrict__ router, long sr, 
     }
     __syncwarp();
     if (groups > 1 && keep < groups) {
-      // Only the `keep` groups of neighbours with the largest choice score stay eligible (ties: the lower group).  A group is
+      // Only the `keep` groups of neighbours with the largest group score stay eligible (ties: the lower group).  A group is
       // dropped when at least `keep` others come before it; its experts count as -inf.  Every lane walks the same groups.
       const int gsz = E / groups;
       for (int g = lane; g < groups; g += 32) {
-        float b = -INFINITY;
-        for (int e = g * gsz; e < (g + 1) * gsz; ++e) b = fmaxf(b, ch[e]);
+        float b = -INFINITY, b2 = -INFINITY;                  // the two largest
+        for (int e = g * gsz; e < (g + 1) * gsz; ++e) {
+          const float c = ch[e];
+          b2 = fmaxf(b2, fminf(b, c));
+          b = fmaxf(b, c);
+        }
+        if (group_sum2 && gsz > 1) b += b2;
         wsel[g] = b;                                          // borrowed: groups <= E
       }
       __syncwarp();
@@ -575,7 +599,10 @@ __global__ void moe_route_all_kernel(const float* __restrict__ router, long sr, 
     const int e = static_cast<int>(idx / ff), c = static_cast<int>(idx - static_cast<long>(e) * ff);
     const float w = wsel[e];
     float v = 0.f;
-    if (w != 0.f) {
+    if (w != 0.f && relu2) {
+      const float up = fmaxf(gu[t * sgu + idx], 0.f);
+      v = w * (up * up);
+    } else if (w != 0.f) {
       const float gt = gu[t * sgu + static_cast<long>(e) * 2 * ff + c], up = gu[t * sgu + static_cast<long>(e) * 2 * ff + ff + c];
       v = w * (gt * sigmoidf_(gt) * up);
     }
@@ -747,7 +774,7 @@ __global__ void embed_streams_kernel(const WT* __restrict__ embed, const int* __
 // input: h1 <- h1 + (previous token's h1 - h1) * mu.
 // ---------------------------------------------------------------------------------------------------------------------
 // A block owns `rows` consecutive tokens; a thread owns fixed columns, so the row buffers in shared memory are thread-private.
-//   x = (x_in or embed[tok]) + o[t] + sum_k y[slot_of[t * top + k]]
+//   x = (x_in or embed[tok]) + o[t] + sum_k wts[t * top + k] y[slot_of[t * top + k]]      (wts null: 1)
 //   x_out = x (float);  raw = x (typed);  h1 = shift(x / rms(x) * w1) (typed);  h2 = x / rms(x) * w2 (typed);  any may be null
 // The previous token's h1 comes from the row above: the block's own, recomputed for the first row of a block, or, for the first
 // token of an entry, the sequence's slot of `state` (zeros at position 0).  The h1 of an entry's last token goes to `carry` [entries, W] and
@@ -759,6 +786,7 @@ struct ParallelBoundary {
   const float* o;
   const float* y;
   const int* slot_of;
+  const float* wts;
   int top;
   const float* w1;
   const float* w2;
@@ -812,9 +840,11 @@ __global__ void __launch_bounds__(256) parallel_boundary_kernel(const ParallelBo
       }
       if (p.y != nullptr) {
         for (int k = 0; k < p.top; ++k) {
-          ldv<V>(p.y + static_cast<long>(p.slot_of[static_cast<long>(t) * p.top + k]) * W + c, a);
+          const long pair = static_cast<long>(t) * p.top + k;
+          const float wk = p.wts != nullptr ? p.wts[pair] : 1.f;
+          ldv<V>(p.y + static_cast<long>(p.slot_of[pair]) * W + c, a);
 #pragma unroll
-          for (int e = 0; e < V; ++e) v[e] += a[e];
+          for (int e = 0; e < V; ++e) v[e] += wk * a[e];
         }
       }
 #pragma unroll
@@ -1131,25 +1161,27 @@ cudaError_t nrl_side_gate(const float* u, long su, const void* table, long st_, 
   return cudaGetLastError();
 }
 
-cudaError_t nrl_swiglu_cols(const float* in, long si, const float* rgate, long srg, void* out, long so, int out_f32, int T, int C,
-                            cudaStream_t s) {
+cudaError_t nrl_swiglu_cols(const float* in, long si, const float* rgate, long srg, float alpha, float limit, float up_shift, void* out, long so,
+                            int out_f32, int T, int C, cudaStream_t s) {
   if (T <= 0 || C <= 0) return cudaSuccess;
+  if (!(limit > 0.f)) return cudaErrorInvalidValue;
+  const GluForm form = {alpha, limit, up_shift};
   if (C % 4 == 0 && si % 4 == 0 && so % 4 == 0 && aligned(in, 16) && aligned(out, out_f32 ? 16 : 8)) {
     const long n4 = static_cast<long>(T) * (C / 4);
     const int blocks4 = static_cast<int>((n4 + 255) / 256 < 148 * 16 ? (n4 + 255) / 256 : 148 * 16);
-    if (out_f32) swiglu_cols_vec4_kernel<float><<<blocks4, 256, 0, s>>>(in, si, rgate, srg, static_cast<float*>(out), so, T, C / 4);
-    else swiglu_cols_vec4_kernel<__nv_bfloat16><<<blocks4, 256, 0, s>>>(in, si, rgate, srg, static_cast<__nv_bfloat16*>(out), so, T, C / 4);
+    if (out_f32) swiglu_cols_vec4_kernel<float><<<blocks4, 256, 0, s>>>(in, si, rgate, srg, form, static_cast<float*>(out), so, T, C / 4);
+    else swiglu_cols_vec4_kernel<__nv_bfloat16><<<blocks4, 256, 0, s>>>(in, si, rgate, srg, form, static_cast<__nv_bfloat16*>(out), so, T, C / 4);
     return cudaGetLastError();
   }
   const long n = static_cast<long>(T) * C;
   const int blocks = static_cast<int>((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
-  if (out_f32) swiglu_cols_kernel<float><<<blocks, 256, 0, s>>>(in, si, rgate, srg, static_cast<float*>(out), so, T, C);
-  else swiglu_cols_kernel<__nv_bfloat16><<<blocks, 256, 0, s>>>(in, si, rgate, srg, static_cast<__nv_bfloat16*>(out), so, T, C);
+  if (out_f32) swiglu_cols_kernel<float><<<blocks, 256, 0, s>>>(in, si, rgate, srg, form, static_cast<float*>(out), so, T, C);
+  else swiglu_cols_kernel<__nv_bfloat16><<<blocks, 256, 0, s>>>(in, si, rgate, srg, form, static_cast<__nv_bfloat16*>(out), so, T, C);
   return cudaGetLastError();
 }
 
 cudaError_t nrl_moe_route_all(const float* router, long sr, const float* correction, int E, int n_real, int top, float route_scale,
-                              int groups, int keep, const float* gu, long sgu, int ff, void* act, long sa, int act_f32, int* ids,
+                              int sigmoid, int groups, int keep, int group_sum2, int relu2, const float* gu, long sgu, int ff, void* act, long sa, int act_f32, int* ids,
                               float* wts, float* self_w, int T, cudaStream_t s) {
   if (T <= 0) return cudaSuccess;
   if (E < 1 || top < 1 || top > E || top > 64 || E > 4096 || n_real < 0 || n_real > E || (n_real < E && self_w == nullptr))
@@ -1158,11 +1190,11 @@ cudaError_t nrl_moe_route_all(const float* router, long sr, const float* correct
   const size_t smem = sizeof(float) * 3 * E;
   const int th = act == nullptr ? 32 : 256;
   if (act_f32)
-    moe_route_all_kernel<float><<<T, th, smem, s>>>(router, sr, correction, E, n_real, top, route_scale, groups, keep, gu, sgu, ff,
-                                                    static_cast<float*>(act), sa, ids, wts, self_w);
+    moe_route_all_kernel<float><<<T, th, smem, s>>>(router, sr, correction, E, n_real, top, route_scale, sigmoid, groups, keep, group_sum2,
+                                                    relu2, gu, sgu, ff, static_cast<float*>(act), sa, ids, wts, self_w);
   else
-    moe_route_all_kernel<__nv_bfloat16><<<T, th, smem, s>>>(router, sr, correction, E, n_real, top, route_scale, groups, keep, gu, sgu,
-                                                            ff, static_cast<__nv_bfloat16*>(act), sa, ids, wts, self_w);
+    moe_route_all_kernel<__nv_bfloat16><<<T, th, smem, s>>>(router, sr, correction, E, n_real, top, route_scale, sigmoid, groups, keep,
+                                                            group_sum2, relu2, gu, sgu, ff, static_cast<__nv_bfloat16*>(act), sa, ids, wts, self_w);
   return cudaGetLastError();
 }
 
@@ -1227,8 +1259,8 @@ cudaError_t nrl_gated_part_rmsnorm(const float* y, long sy, const float* gate, l
 }
 
 cudaError_t nrl_parallel_boundary(const float* x_in, const void* embed, int w_f32, const int* tok, const float* o, const float* y,
-                                  const int* slot_of, int top, const float* w1, const float* w2, const float* mu, float eps, float* x_out,
-                                  void* raw, void* h1, void* h2, int h_f32, const int* cu, const int* tok_entry, const int* start,
+                                  const int* slot_of, const float* wts, int top, const float* w1, const float* w2, const float* mu, float eps,
+                                  float* x_out, void* raw, void* h1, void* h2, int h_f32, const int* cu, const int* tok_entry, const int* start,
                                   const int* state_slot, const float* state, float* carry, const float* commit, float* commit_state, int T,
                                   int W, cudaStream_t s) {
   if (T <= 0) return cudaSuccess;
@@ -1240,7 +1272,7 @@ cudaError_t nrl_parallel_boundary(const float* x_in, const void* embed, int w_f3
     return cudaErrorInvalidValue;
   // tokens per block: one while that fills the GPU, up to six (the row above a block is read once more per block)
   const int rows = T >= 8192 ? 6 : T >= 4096 ? 4 : T >= 2048 ? 3 : 1;
-  const ParallelBoundary p = {x_in, embed, tok, o, y, slot_of, top, w1, w2, mu, eps, x_out, raw, h1, h2, cu, tok_entry, start, state_slot,
+  const ParallelBoundary p = {x_in, embed, tok, o, y, slot_of, wts, top, w1, w2, mu, eps, x_out, raw, h1, h2, cu, tok_entry, start, state_slot,
                               state, carry, commit, commit_state, T, W, rows};
   auto ok = [](const void* q, size_t a) { return q == nullptr || aligned(q, a); };
   const size_t ha = h_f32 ? 16 : 8;

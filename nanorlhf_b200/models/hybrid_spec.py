@@ -20,7 +20,7 @@ from .hf_io import load_state_dict, save_state_dict
 @dataclass
 class MixerSpec:
     """One token mixer of a layer.  ``kind``: window_attention | conv_attention | ssd | gated_delta | latent_attention | gla |
-    rot_attention | mlstm.  ``prefix``: tensor-name prefix."""
+    rot_attention | mlstm | lightning.  ``prefix``: tensor-name prefix."""
     kind: str
     prefix: str
     out_scale: float = 1.0
@@ -49,7 +49,8 @@ class MixerSpec:
     rot_dims: int = 0            # how many of the rot_dim columns turn (the rest pass unchanged)
     rot_base: float = 10000.0    # frequency i of rot_dims / 2 is rot_base^(-2 i / rot_dims)
     rot_layout: str = "interleaved"   # "interleaved": column 2i turns with 2i + 1;  "half": i with i + rot_dims / 2
-    rot_scaling: Optional[dict] = None  # frequency-dependent stretch {"factor", "original", "fast", "slow"} with its cos / sin multiplier
+    rot_scaling: Optional[dict] = None  # frequency-dependent stretch: {"factor", "original", "fast", "slow"} (linear in the pair index, with a cos /
+                                 # sin multiplier) or {"factor", "original", "low", "high"} (linear in the turns within `original` positions)
     head_sink: bool = False      # the softmax denominator also holds exp(sink_h) (tensor "sink"): a score with no key and no value
     # gla (gated linear attention, S = diag(decay) S + k v^T, o = S^T q D^-1/2; decay = sigmoid(a2 (a1 h) + a2.b)^(1 / tau) per key channel):
     tau: float = 1.0
@@ -73,6 +74,9 @@ class MixerSpec:
     # m' = max(f + m, i); S = exp(f + m - m') S + exp(i - m') k v^T, n likewise with k; o = S^T q / (max(|n . q|, exp(-m')) + 1e-6) with
     # q scaled by dim^-1/2; per-head RMS norm, weight "norm", sigmoid gate "g"):
     gate_cap: float = 0.0
+    # lightning (linear attention with a constant decay per head: q, k, v = silu of their projections; S = decay_h S + k v^T, o = S^T q; RMS norm in
+    # `norm_groups` parts of the concatenated heads, weight "norm", sigmoid gate "g"):
+    decay: tuple = ()
 
 
 @dataclass
@@ -80,20 +84,26 @@ class LayerSpec:
     index: int
     mixers: List[MixerSpec]
     ff: int = 0                  # 0: no feed-forward; else its inner width (of one expert for "moe")
-    ff_act: str = "relu2"        # "relu2": W_down relu(W_up h)^2;  "swiglu": W_down (silu(W_gate h) * W_up h)
+    ff_act: str = "relu2"        # "relu2": W_down relu(W_up h)^2;  "swiglu": W_down (g sigmoid(ff_alpha g) * (u + ff_up_shift)), g = W_gate h,
+                                 # u = W_up h; ff_limit > 0 (dense only) caps g from above and u on both sides first
+    ff_alpha: float = 1.0
+    ff_up_shift: float = 0.0
+    ff_limit: float = 0.0
     ff_kind: str = "dense"       # "dense" | "moe" (experts e0.., top-k router)
     experts: int = 0
     top: int = 0
     route: str = "softmax_top"   # "softmax_top": the largest logits (+ bias "router.b"), weights = softmax over the chosen logits
                                  # "softmax_all": scores = softmax over all router outputs, chosen by score + "correction",
                                  #                weights = the chosen scores / their sum * route_scale
+                                 # "sigmoid_all": the same with scores = sigmoid of each router output
                                  # "sigmoid": scores = sigmoid of the logits, the largest are chosen, weights = the chosen scores
     weight_input: bool = False   # "softmax_top" / "sigmoid": the weight multiplies the expert's input instead of its result
     route_scale: float = 1.0
-    route_groups: int = 1        # "softmax_all": > 1: the router outputs form that many equal groups of neighbours and only experts of the
-    route_keep: int = 1          # `route_keep` groups with the largest choice score can be chosen
+    route_groups: int = 1        # "softmax_all" / "sigmoid_all": > 1: the router outputs form that many equal groups of neighbours and only experts of
+    route_keep: int = 1          # the `route_keep` groups with the largest group score can be chosen
+    group_score: str = "max"     # a group's score: its largest choice score, or the sum of its two largest ("top2")
     identity_experts: int = 0    # router outputs behind the `experts` real ones whose expert returns its input
-    shared_ff: int = 0           # > 0: a SwiGLU expert of this width for every token (tensors "shared.*")
+    shared_ff: int = 0           # > 0: an expert of this width (activation ff_act) for every token (tensors "shared.*")
     shared_gate: bool = False    # its result times sigmoid(shared.sg h), one number per token
     side_dim: int = 0            # > 0: per-layer token input after the feed-forward (stream kind "post_norm"): columns
                                  # [index * side_dim, (index + 1) * side_dim) of the table "side.embed", gated by gelu_tanh(side.gate x),
@@ -113,7 +123,7 @@ class StreamSpec:
     the start); sublayer q of a layer reads ``layernorm(sum_s hc<q>.in[s] x_s)`` (weight norm<q>, bias norm<q>.b) and every stream becomes
     ``x_t <- sum_s hc<q>.mix[s, t] x_s + hc<q>.out[t] y``; the output reads the layer norm of the streams' sum (``hyper_weights`` False:
     one stream with the plain residual sum, no hc tensors).  ``kind`` "parallel": ``x += mixer(norm1(x)) + ff(norm2(x))``, both of the same
-    x; ``token_shift``: the mixer reads ``h + (h_prev - h) * shift`` with ``h = norm1(x)`` and ``h_prev`` the previous token's h (zeros for the
+    x; ``shared_norm``: there is no norm2, both read norm1(x); ``token_shift``: the mixer reads ``h + (h_prev - h) * shift`` with ``h = norm1(x)`` and ``h_prev`` the previous token's h (zeros for the
     first; tensor "shift").
 
     ``loop`` (start, stop, times): layers start .. stop - 1 run that many times in a row with the same weights, every pass with cache
@@ -130,6 +140,7 @@ class StreamSpec:
     streams: int = 1                            # "hyper": copies of the residual stream
     hyper_weights: bool = True                  # "hyper": the layers carry hc1 / hc2 tensors
     token_shift: bool = False                   # "parallel"
+    shared_norm: bool = False                   # "parallel": mixer and feed-forward read the same norm
     centred_norm: bool = False                  # "parallel": norm weights are stored around zero (the norm multiplies by 1 + w)
     loop: Optional[tuple] = None                # "parallel": (start, stop, times)
     tied_head: bool = False                     # logits = embed x (the table itself, without embed_scale); no "head" tensor

@@ -1,5 +1,5 @@
 """Op layer of hybrid (attention + recurrent-state) decoders: thin, launch-counting wrappers over the sm_100a kernels of
-``csrc/stream_ops.cu``, ``csrc/recurrent.cu``, ``csrc/attention_window.cu`` / ``attention_window_mma.cu`` /
+``csrc/stream_ops.cu``, ``csrc/recurrent.cu``, ``csrc/lightning.cu``, ``csrc/attention_window.cu`` / ``attention_window_mma.cu`` /
 ``attention_latent_mma.cu`` and ``csrc/moe.cu``
 (with the grouped form of ``csrc/gemm_tc.cu``).
 
@@ -81,7 +81,7 @@ def window_attention(q, k_cache, v_cache, plan, window, scale, out_scale, out, i
     """``impl``: "auto" (tensor cores for prompt portions over bf16 pages, the scalar tile kernel otherwise) or one kernel by
     name; a kernel that does not fit the shapes raises.  ``chunked``: keys of the query's own chunk of ``window`` positions
     instead of the last ``window`` keys.  ``head_scale`` / ``head_slope`` [heads]: per-head score multiplier and linear distance
-    penalty; ``gate`` [T, heads]: the head's output is multiplied by sigmoid(gate); ``head_sink`` [heads]: the softmax denominator
+    penalty; ``gate`` [T, heads] or [T, heads * value size]: the head's output (or every column) is multiplied by sigmoid(gate); ``head_sink`` [heads]: the softmax denominator
     also holds exp(sink).  ``value_size`` > 0 (with ``v_cache is k_cache``): the values are the first ``value_size`` columns of the
     key rows (latent attention: one cached row per token serves as key and value of every head); ``q`` may then be head-major
     [heads, T, >= D], the layout a batched GEMM leaves.  ``softcap`` > 0: the scaled score becomes softcap * tanh(score / softcap);
@@ -131,7 +131,7 @@ def interleave_gate_up(gate, up):
 
 
 def moe_grouped_ffn(h, ids, wts, w_gate_up, w_down, experts, ff, out, fused_act: bool = False, identity: int = 0,
-                    weight_input: bool = False):
+                    weight_input: bool = False, relu2: bool = False):
     """Expert feed-forwards of a routed batch on the grouped tcgen05 GEMM.  ``h`` bf16 [T, W]; ``ids`` / ``wts`` [T, top] from
     ``moe_route``; ``w_gate_up`` bf16 [experts * 2 ff, W] (per expert its gate rows, then its up rows; ``fused_act``: interleaved
     per 32 features by ``interleave_gate_up``, the SwiGLU is then formed in the GEMM's epilogue); ``w_down`` bf16
@@ -140,18 +140,21 @@ def moe_grouped_ffn(h, ids, wts, w_gate_up, w_down, experts, ff, out, fused_act:
     skipped (the caller adds their share of the input).
     ``weight_input``: the weight multiplies the expert's INPUT: the gate and up products are scaled per row before the activation
     (the projections have no bias).  ``out`` is then not written; returns ``(y, slot_of)``, the experts' results in expert order and
-    each (token, choice) pair's row, for a boundary kernel that sums them."""
+    each (token, choice) pair's row, for a boundary kernel that sums them.  ``out`` None: the same, the weights are left to that kernel.
+    ``relu2``: experts without a gate, ``w_gate_up`` bf16 [experts * ff, W]; the squared ReLU is formed in the GEMM's epilogue."""
     import torch
     T, W = h.shape
     R = ids.numel()
     ext = _ext()
-    native._count(5 if fused_act else 6)
+    native._count(5 if fused_act or relu2 else 6)
     rw = torch.empty(R, dtype=torch.float32, device=h.device) if weight_input else None
     slot_of, row_token, _seg, tiles, num_tiles = ext.moe_plan(ids, experts + identity, 128, experts, wts if weight_input else None, rw)
     xp = torch.empty(R, W, dtype=h.dtype, device=h.device)
     ext.gather_rows(h, row_token, xp)
     act = torch.empty(R, ff, dtype=h.dtype, device=h.device)
-    if fused_act:
+    if relu2:
+        ext.gemm_tc_grouped(xp, w_gate_up, None, tiles, num_tiles, 0, act, rw, True)
+    elif fused_act:
         ext.gemm_tc_grouped(xp, w_gate_up, None, tiles, num_tiles, 0, act, rw)
     else:
         gu = torch.empty(R, 2 * ff, dtype=torch.float32, device=h.device)
@@ -159,7 +162,7 @@ def moe_grouped_ffn(h, ids, wts, w_gate_up, w_down, experts, ff, out, fused_act:
         ext.swiglu_rows(gu, act, rw)
     y = torch.empty(R, W, dtype=torch.float32, device=h.device)
     ext.gemm_tc_grouped(act, w_down, y, tiles, num_tiles)
-    if weight_input:
+    if weight_input or out is None:
         native._count(-1)
         return y, slot_of
     ext.moe_combine(y, slot_of, wts, out)
@@ -185,19 +188,22 @@ def side_gate(u, table, col0, tok, out, dim):
     _ext().side_gate(u, table, col0, tok, out, dim)
 
 
-def swiglu_cols(gu, row_gate, out):
-    """out = silu(gu[:, :C]) * gu[:, C:] (``* sigmoid(row_gate)`` [T, 1] when given)."""
+def swiglu_cols(gu, row_gate, out, alpha: float = 1.0, limit: float = 0.0, up_shift: float = 0.0):
+    """out = g sigmoid(alpha g) * (u + up_shift) with g = gu[:, :C], u = gu[:, C:] (``* sigmoid(row_gate)`` [T, 1] when given); ``limit`` > 0 caps
+    g from above and u on both sides first.  The defaults are SwiGLU."""
     native._count()
-    _ext().swiglu_cols(gu, row_gate, out)
+    _ext().swiglu_cols(gu, row_gate, out, alpha, limit if limit > 0 else float("inf"), up_shift)
 
 
 def moe_route_all(router, correction, n_real, top, scale, gu=None, ff=0, act=None, ids=None, wts=None, self_w=None, groups: int = 1,
-                  keep: int = 1):
-    """Routing by a softmax over all router outputs (the last ``E - n_real`` are identity experts), choice by score + correction,
+                  keep: int = 1, sigmoid: bool = False, group_score: str = "max", relu2: bool = False):
+    """Routing by a softmax over all router outputs (``sigmoid``: each output's own sigmoid; the last ``E - n_real`` are identity experts), choice by score + correction,
     weights = chosen scores / their sum * scale; ``self_w`` [T] receives the identity experts' weights.  ``groups`` > 1: the outputs
-    form that many equal groups of neighbours and only the ``keep`` groups with the largest choice score can be chosen from."""
+    form that many equal groups of neighbours and only the ``keep`` groups with the largest score can be chosen from; ``group_score``:
+    a group's largest choice score ("max") or the sum of its two largest ("top2").  ``relu2``: the dense form's experts have no gate."""
     native._count()
-    _ext().moe_route_all(router, correction, n_real, top, scale, groups, keep, gu, ff, act, ids, wts, self_w)
+    _ext().moe_route_all(router, correction, n_real, top, scale, groups, keep, gu, ff, act, ids, wts, self_w, sigmoid,
+                         {"max": False, "top2": True}[group_score], relu2)
 
 
 def gla_prep(qkv, a_raw, a_bias, tau, decay, heads, dim):
@@ -215,7 +221,9 @@ def latent_kv_write(q, heads, dim, rot_dim, dkv, norm_w, eps, freq, rot_dims, mu
 
 
 def rotary_frequencies(dims: int, base: float, scaling=None):
-    """(frequencies [dims / 2] as float64 list, cos / sin multiplier).  ``scaling`` {"factor", "original", "fast", "slow"}: frequencies
+    """(frequencies [dims / 2] as float64 list, cos / sin multiplier).  ``scaling`` {"factor", "original", "low", "high"}: frequencies that turn
+    more than ``high`` times within ``original`` positions keep their value, those that turn less than ``low`` times are divided by ``factor``,
+    between the two the value moves linearly in the number of turns (multiplier 1).  {"factor", "original", "fast", "slow"}: frequencies
     that turn more than ``fast`` times within ``original`` positions keep their value, those that turn less than ``slow`` times
     are divided by ``factor``, linear in the pair index between; cos and sin are then multiplied by 0.1 ln(factor) + 1."""
     import math
@@ -223,6 +231,17 @@ def rotary_frequencies(dims: int, base: float, scaling=None):
     if not scaling:
         return f, 1.0
     factor, orig = float(scaling["factor"]), float(scaling["original"])
+    if "low" in scaling:
+        low, high = float(scaling["low"]), float(scaling["high"])
+        out = []
+        for fi in f:
+            turns = orig * fi / (2.0 * math.pi)
+            if turns > high or turns < low:
+                out.append(fi if turns > high else fi / factor)
+            else:
+                s = (turns - low) / (high - low) if high > low else 1.0
+                out.append((1.0 - s) * fi / factor + s * fi)
+        return out, 1.0
 
     def pair_of(turns):                                    # the (real-valued) pair index that turns `turns` times in `orig` positions
         return dims * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
@@ -236,14 +255,14 @@ def rotary_frequencies(dims: int, base: float, scaling=None):
 
 
 def parallel_boundary(plan, embed, eps, x_in=None, o=None, y=None, slot_of=None, w1=None, w2=None, mu=None, x_out=None, raw=None, h1=None,
-                      h2=None, state=None, carry=None, commit=None, commit_state=None):
-    """Boundary of a stream whose mixer and feed-forward read the same x: ``x = (x_in or embed[tokens]) + o + sum_k y[slot_of]`` goes to
+                      h2=None, state=None, carry=None, commit=None, commit_state=None, wts=None):
+    """Boundary of a stream whose mixer and feed-forward read the same x: ``x = (x_in or embed[tokens]) + o + sum_k wts y[slot_of]`` (``wts`` None: 1) goes to
     ``x_out`` (float) and ``raw`` (operand type); ``h1 = rmsnorm(x) * w1`` (with ``mu``: moved towards the previous token's row, which an
     entry's first token finds in its slot of ``state``) and ``h2 = rmsnorm(x) * w2``.  ``carry`` [entries, W] receives the rows that
     later steps need; the next boundary hands them over (``commit`` -> ``commit_state``)."""
     native._count()
     _ext().parallel_boundary(x_in, embed, plan.tokens, o, y, slot_of, w1, w2, mu, eps, x_out, raw, h1, h2, plan.cu, plan.tok_entry,
-                             plan.start, plan.state_slot, state, carry, commit, commit_state)
+                             plan.start, plan.state_slot, state, carry, commit, commit_state, wts)
 
 
 def gate_cols(x, gate, scale, out):
@@ -270,6 +289,25 @@ def hyper_boundary(xs, o, o_bias, self_w, mix, outw, inw, ln_w, ln_b, eps, h):
     With ``h``: ``u = sum_s inw[s] x_s`` (``inw`` None: the plain sum) and ``h = layernorm(u) * ln_w + ln_b`` in the operand type."""
     native._count()
     _ext().hyper_boundary(xs, o, o_bias, self_w, mix, outw, inw, ln_w, ln_b, eps, h)
+
+
+LIGHTNING_IMPLS = {"auto": 0, "registers": 1, "global": 2, "chunk": 3}
+LIGHTNING_CHUNK = 64
+
+
+def decay_powers(decay, device):
+    """float [heads, LIGHTNING_CHUNK + 1]: decay_h^n for n = 0 .. LIGHTNING_CHUNK, formed in float64."""
+    import torch
+    d = torch.tensor([float(x) for x in decay], dtype=torch.float64)[:, None]
+    return (d ** torch.arange(LIGHTNING_CHUNK + 1, dtype=torch.float64)[None, :]).to(device=device, dtype=torch.float32).contiguous()
+
+
+def lightning_scan(qkv, col_q, col_k, col_v, pows, state, o, plan, chunk_ok: bool, impl: str = "auto"):
+    """Linear attention with a constant decay per head over raw projections (silu is applied to q, k and v here): ``S = decay_h S + k v^T``,
+    ``o = S^T q``; ``state`` float [slots, heads, D, Dv].  ``chunk_ok``: long portions may run in chunks on the tensor cores (bf16 operands,
+    float state)."""
+    native._count(2 if impl == "chunk" or (impl == "auto" and chunk_ok and plan.T != plan.E) else 1)
+    _ext().lightning_scan(qkv, col_q, col_k, col_v, pows, state, o, plan.cu, plan.start, plan.state_slot, chunk_ok, LIGHTNING_IMPLS[impl])
 
 
 MLSTM_IMPLS = {"auto": 0, "column": 1, "global": 2}

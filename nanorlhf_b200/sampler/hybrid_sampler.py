@@ -31,6 +31,9 @@ step in a per-sequence slot) and it gives chunked prefill and continuous batchin
   times in a row with shared weights and a projection of [x; embedding] in front of every pass, each pass with pages and state of
   its own; its latent attention may form queries through a normed latent and gate the heads element by element; its router weighs
   the experts' inputs with sigmoid scores;
+* a parallel stream may also feed mixer and feed-forward from one norm: all their projections are then one GEMM in and one GEMM out, and
+  the boundary gathers the weighted expert rows; its linear attention with a constant decay per head runs prompt portions in chunks on
+  the tensor cores;
 * the residual stream, its depth-weighted average, norms, scores, softmax, decays and recurrent state are float32 in both
   serving modes; ``dtype="bf16"`` keeps GEMM operands and KV pages in bf16 (fp32 accumulation, fp32 GEMM results),
   ``dtype="fp32"`` keeps everything in float32 with TF32 off;
@@ -188,11 +191,11 @@ class HybridSampler:
                     if st.hyper_weights:
                         L.hc_in, L.hc_out, L.hc_mix = (self._f(f"{p}hc{n}.{x}") for x in ("in", "out", "mix"))
                     self.layers.append(L)
-            elif st.kind == "parallel":                   # one stage per layer; its feed-forward reads an operand of its own (L.ff)
-                L = self._build_stage(spec, spec.mixers, False)
+            elif st.kind == "parallel":                   # one stage per layer; its feed-forward reads an operand of its own (L.ff) or the same one
+                L = self._build_stage(spec, spec.mixers, st.shared_norm)
                 L.w_pre = self._norm_gain(p + "norm1")
                 L.shift = self._f(p + "shift") if st.token_shift else None
-                if spec.ff:
+                if spec.ff and not st.shared_norm:
                     self._attach_feed_forward(L, spec)
                     L.ff.w_pre = self._norm_gain(p + "norm2")
                 self.layers.append(L)
@@ -407,12 +410,21 @@ class HybridSampler:
                 pad_in()
                 for n in ("i.b", "f.b", "norm"):
                     M.vec[n] = self._f(q + n)
+            elif ms.kind == "lightning":
+                pad_in()                                   # q, k and v start on 32-byte boundaries when the head sizes allow
+                for n in ("q", "k", "v", "g"):
+                    M.cols[n] = add_in(q + n)
+                pad_in()
+                M.vec["norm"] = self._f(q + "norm")
+                M.vec["pows"] = hy.decay_powers(ms.decay, dev)
             else:
                 raise ValueError(f"unknown mixer kind {ms.kind!r}")
             M.out_col, M.out_size = add_out(q + "o")
             L.mixers.append(M)
         L.ff_col = L.ff_out_col = None
         if with_ff and spec.ff:
+            if mixer_specs:
+                pad_in()
             if spec.ff_kind == "dense" and spec.ff_act == "swiglu":      # [gate rows | up rows]
                 c0 = add_in(p + "mlp.gate")[0]
                 add_in(p + "mlp.up")
@@ -426,7 +438,9 @@ class HybridSampler:
                 # grouped GEMM, [experts * 2 ff, W] (gate rows, then up rows) and [experts * W, ff]
                 L.router_col = add_in(p + "mlp.router")
                 L.router_bias = self._router_vector(spec, p)
-                if spec.ff % 32 == 0:                      # gate / up rows interleaved: the SwiGLU is formed in the GEMM's epilogue
+                if spec.ff_act == "relu2":                 # no gate: [experts * ff, W], the activation in the GEMM's epilogue
+                    L.w_gate_up = torch.cat([self._t(f"{p}mlp.e{e}.up").to(device=dev, dtype=wd) for e in range(spec.experts)], 0).contiguous()
+                elif spec.ff % 32 == 0:                      # gate / up rows interleaved: the SwiGLU is formed in the GEMM's epilogue
                     L.w_gate_up = torch.cat([hy.interleave_gate_up(self._t(f"{p}mlp.e{e}.gate").to(device=dev, dtype=wd),
                                                                    self._t(f"{p}mlp.e{e}.up").to(device=dev, dtype=wd))
                                              for e in range(spec.experts)], 0).contiguous()
@@ -439,7 +453,8 @@ class HybridSampler:
                 L.router_bias = self._router_vector(spec, p)
                 c0 = n_in
                 for e in range(spec.experts):
-                    add_in(f"{p}mlp.e{e}.gate")
+                    if spec.ff_act == "swiglu":
+                        add_in(f"{p}mlp.e{e}.gate")
                     add_in(f"{p}mlp.e{e}.up")
                 L.ff_col = (c0, n_in - c0)
                 c0 = k_out
@@ -450,9 +465,11 @@ class HybridSampler:
                 raise ValueError(f"unknown feed-forward kind {spec.ff_kind!r}")
             if spec.ff_kind == "moe" and spec.shared_ff:     # an expert for every token: rides in the fused matrices like a dense one
                 pad_in()
-                c0 = add_in(p + "mlp.shared.gate")[0]
+                c0 = n_in
+                if spec.ff_act == "swiglu":
+                    add_in(p + "mlp.shared.gate")
                 add_in(p + "mlp.shared.up")
-                L.shared_col = (c0, 2 * spec.shared_ff)
+                L.shared_col = (c0, n_in - c0)
                 if spec.shared_gate:
                     L.sg_col = add_in(p + "mlp.shared.sg")
                 L.shared_out_col = add_out(p + "mlp.shared.down")
@@ -474,7 +491,7 @@ class HybridSampler:
 
     def _router_vector(self, spec, p):
         """The vector added to the router's outputs before the choice: a bias on the logits, or a correction of the scores."""
-        name = p + ("mlp.correction" if spec.route == "softmax_all" else "mlp.router.b")
+        name = p + ("mlp.correction" if spec.route in ("softmax_all", "sigmoid_all") else "mlp.router.b")
         return self._f(name) if self.lm.has_tensor(name) else None
 
     def _moe_grouped(self, spec) -> bool:
@@ -528,7 +545,7 @@ class HybridSampler:
                     M.conv_state = torch.zeros(num_slots, ms.conv - 1, ch, **f32)
                 elif ms.kind == "latent_attention":       # one row per token: [normed latent | rotated shared key part]
                     M.k_cache = torch.zeros(n, 1, self.PAGE, ms.kv_rank + ms.rot_dim, dtype=wd, device=dev)
-                elif ms.kind == "gla":
+                elif ms.kind in ("gla", "lightning"):
                     M.state = torch.zeros(num_slots, ms.heads, ms.dim, ms.vdim, **f32)
                 elif ms.kind == "rot_attention":
                     if M.owns_kv:                          # every score map has key heads of its own; the values are shared by the maps
@@ -647,6 +664,8 @@ class HybridSampler:
                 self._rot_attention(M, U, plan, eps, out)
             elif kind == "mlstm":
                 self._mlstm(M, U, plan, eps, out)
+            elif kind == "lightning":
+                self._lightning(M, U, plan, eps, out)
             elif kind == "conv_attention":
                 self._conv_attention(M, U, plan, out, ctx, L.spec.index)
             elif kind == "gated_delta":
@@ -676,8 +695,7 @@ class HybridSampler:
                 (c, n), (oc, on) = L.side_col, L.side_out_col
                 hy.side_gate(U[:, c:c + n], self.side_table, L.side_col0, plan.tokens, A[:, oc:oc + on], n)
             if L.shared_col is not None:
-                (c, n), (oc, on) = L.shared_col, L.shared_out_col
-                hy.swiglu_cols(U[:, c:c + n], U[:, L.sg_col[0]:L.sg_col[0] + 1] if L.sg_col is not None else None, A[:, oc:oc + on])
+                self._shared_expert(L, U, A)
             if L.ff_col is not None:
                 self_w = self._feed_forward(L, U, A)
             o = self._mm(A, L.w_out) if L.k_out else None                             # [T, W] float
@@ -742,36 +760,40 @@ class HybridSampler:
         if self.stream.loop:
             hy.parallel_boundary(plan, self.embed, eps, raw=raw)
             z0 = self._mm(raw, self.w_pass_x0)
-        x = o = y = slot_of = None                         # x None: the embedding
+        x = o = y = slot_of = wts = None                   # x None: the embedding
         done = {}                                          # what the last token-shifted boundary left for its state
         for i, L in enumerate(self.layers):
             if L.pass_entry:                               # x = loop.in [x; x0], the second half already multiplied
                 if i:                                      # (in front of layer 0 ``raw`` holds the embedding already)
-                    hy.parallel_boundary(plan, self.embed, eps, x_in=x, o=o, y=y, slot_of=slot_of, raw=raw,
+                    hy.parallel_boundary(plan, self.embed, eps, x_in=x, o=o, y=y, slot_of=slot_of, wts=wts, raw=raw,
                                          x_out=xs[i & 1] if keep is not None else None, **done)
                 if keep is not None and i:
                     keep.append(xs[i & 1].clone())
-                x, o, y, slot_of, done = self._mm(raw, self.w_pass_x), z0, None, None, {}
+                x, o, y, slot_of, wts, done = self._mm(raw, self.w_pass_x), z0, None, None, None, {}
             F, xn = L.ff, xs[i & 1]
             carry = carries[i & 1] if L.shift is not None else None
-            hy.parallel_boundary(plan, self.embed, eps, x_in=x, o=o, y=y, slot_of=slot_of, w1=L.w_pre, mu=L.shift, x_out=xn, h1=h1,
+            hy.parallel_boundary(plan, self.embed, eps, x_in=x, o=o, y=y, slot_of=slot_of, wts=wts, w1=L.w_pre, mu=L.shift, x_out=xn, h1=h1,
                                  w2=F.w_pre if F is not None else None, h2=h2 if F is not None else None, state=L.shift_state, carry=carry,
                                  **done)
             done = dict(commit=carry, commit_state=L.shift_state) if carry is not None else {}
             if keep is not None and i and not L.pass_entry:
                 keep.append(xn.clone())
-            x, y, slot_of = xn, None, None
+            x, y, slot_of, wts = xn, None, None, None
             U = self._mm(h1, L.w_in)                                                  # [T, n_in] float
             A = (torch.zeros if L.out_pad else torch.empty)(T, L.k_out, dtype=wd, device=dev)
             self._run_mixers(L, U, A, plan, eps)
-            if F is not None:
-                U = self._mm(h2, F.w_in)
-                if F.ff_col is not None:
-                    self._feed_forward(F, U, A)
-                if F.w_gate_up is not None:
-                    y, slot_of = self._experts_grouped(F, U, h2, None)
+            hf = h1
+            if F is not None:                              # the feed-forward reads a norm (and a GEMM) of its own
+                U, hf = self._mm(h2, F.w_in), h2
+            F = F or L
+            if F.shared_col is not None:
+                self._shared_expert(F, U, A)
+            if F.ff_col is not None:
+                self._feed_forward(F, U, A)
+            if F.w_gate_up is not None:
+                y, slot_of, wts = self._experts_grouped(F, U, hf, None, rows_out=True)
             o = self._mm(A, L.w_out)                                                  # [T, W] float
-        hy.parallel_boundary(plan, self.embed, eps, x_in=x, o=o, y=y, slot_of=slot_of, w1=self.final_gain, h1=h1,
+        hy.parallel_boundary(plan, self.embed, eps, x_in=x, o=o, y=y, slot_of=slot_of, wts=wts, w1=self.final_gain, h1=h1,
                              x_out=xs[len(self.layers) & 1] if keep is not None else None, **done)
         if keep is not None:
             keep.append(xs[len(self.layers) & 1].clone())
@@ -809,9 +831,7 @@ class HybridSampler:
                                 keep_first=ms.keep_first, dist_bias=M.vec.get("rel"), v_div=2)
             hy.diff_combine(a, M.lam, 1.0 - ms.diff, eps, gate, ms.out_scale, out, ms.heads, ms.kv_heads)
             return
-        if gate is not None:
-            raise NotImplementedError("an element-wise output gate goes with two score maps")
-        hy.window_attention(q, M.k_cache, M.v_cache, plan, window, ms.scale, ms.out_scale, out, head_sink=M.vec.get("sink"),
+        hy.window_attention(q, M.k_cache, M.v_cache, plan, window, ms.scale, ms.out_scale, out, gate=gate, head_sink=M.vec.get("sink"),
                             softcap=ms.softcap, keep_first=ms.keep_first, dist_bias=M.vec.get("rel"))
 
     def _mlstm(self, M, U, plan, eps, out):
@@ -825,6 +845,16 @@ class HybridSampler:
                       ms.gate_cap, ms.dim ** -0.5, M.state, M.aux_state, o, m, plan)
         cg, ng = M.cols["g"]
         hy.mlstm_out(o, m, U[:, cg:cg + ng], M.vec["norm"], eps, ms.out_scale, out, ms.heads)
+
+    def _lightning(self, M, U, plan, eps, out):
+        """Linear attention with a constant decay per head: the scan reads the raw projections where the fused GEMM left them (portions in
+        chunks on the tensor cores when operands are bf16); a second launch norms, weights and gates."""
+        ms = M.spec
+        nv = ms.heads * ms.vdim
+        o = torch.empty(plan.T, nv, dtype=torch.float32, device=U.device)
+        hy.lightning_scan(U, M.cols["q"][0], M.cols["k"][0], M.cols["v"][0], M.vec["pows"], M.state, o, plan, not self.fp32)
+        cg, ng = M.cols["g"]
+        hy.gated_part_rmsnorm(o, U[:, cg:cg + ng], M.vec["norm"], nv // ms.norm_groups, "sigmoid", False, eps, ms.out_scale, out)
 
     def _latent_attention(self, M, U, plan, eps, out):
         """Latent attention in its absorbed form.  The cache holds one row [latent | rotated shared key part] per token; a head's
@@ -949,50 +979,68 @@ class HybridSampler:
             logits.mul_(st.logit_scale)
         return logits[:, :cfg.vocab]                      # rows keep their padded (16-byte aligned) stride
 
-    def _experts_grouped(self, L, U, h, o, want_self: bool = False):
+    def _experts_grouped(self, L, U, h, o, want_self: bool = False, rows_out: bool = False):
         """Route, then run only the chosen experts: rows sorted by expert through two grouped GEMMs.  ``want_self``: also return the
-        per-token weight of the chosen identity experts (None without such experts).  Experts whose input is weighed return their
-        rows in expert order and every (token, choice) pair's row instead of the sum."""
+        per-token weight of the chosen identity experts (None without such experts).  ``rows_out``: return the experts' rows in
+        expert order, every (token, choice) pair's row and its weight (None: already spent on the expert's input) instead of the sum."""
         spec = L.spec
         T, dev = h.shape[0], h.device
         rc, E = L.router_col
         ids = torch.empty(T, spec.top, dtype=torch.int32, device=dev)
         wts = torch.empty(T, spec.top, dtype=torch.float32, device=dev)
         self_w = None
-        if spec.route == "softmax_all":
+        if spec.route in ("softmax_all", "sigmoid_all"):
             if spec.identity_experts:
                 self_w = torch.empty(T, dtype=torch.float32, device=dev)
             hy.moe_route_all(U[:, rc:rc + E], L.router_bias, spec.experts, spec.top, spec.route_scale, ids=ids, wts=wts, self_w=self_w,
-                             groups=spec.route_groups, keep=spec.route_keep)
+                             groups=spec.route_groups, keep=spec.route_keep, sigmoid=spec.route == "sigmoid_all",
+                             group_score=spec.group_score)
         else:
             hy.moe_route(U[:, rc:rc + E], L.router_bias, spec.top, ids=ids, wts=wts, sigmoid=spec.route == "sigmoid")
-        if spec.weight_input:                              # the weights are spent inside: what is left is a sum of rows
-            return hy.moe_grouped_ffn(h, ids, wts, L.w_gate_up, L.w_down, spec.experts, spec.ff, None, fused_act=spec.ff % 32 == 0,
-                                      weight_input=True)
+        relu2 = spec.ff_act == "relu2"
+        fused = not relu2 and spec.ff % 32 == 0
+        if rows_out:                                       # what is left is a (weighted) sum of rows
+            if spec.identity_experts:
+                raise NotImplementedError("identity experts go with a combined result")
+            y, slot_of = hy.moe_grouped_ffn(h, ids, wts, L.w_gate_up, L.w_down, spec.experts, spec.ff, None, fused_act=fused,
+                                            weight_input=spec.weight_input, relu2=relu2)
+            return y, slot_of, None if spec.weight_input else wts
+        if spec.weight_input:
+            raise NotImplementedError("experts whose input is weighed go with a stream that sums their rows")
         y = torch.empty(T, self.cfg.width, dtype=torch.float32, device=dev)
-        hy.moe_grouped_ffn(h, ids, wts, L.w_gate_up, L.w_down, spec.experts, spec.ff, y, fused_act=spec.ff % 32 == 0,
-                           identity=spec.identity_experts)
+        hy.moe_grouped_ffn(h, ids, wts, L.w_gate_up, L.w_down, spec.experts, spec.ff, y, fused_act=fused, identity=spec.identity_experts,
+                           relu2=relu2)
         if o is not None:
             native._count()
             y = o.add_(y)
         return (y, self_w) if want_self else y
 
+    def _shared_expert(self, L, U, A):
+        (c, n), (oc, on) = L.shared_col, L.shared_out_col
+        if L.spec.ff_act == "relu2":
+            if L.sg_col is not None:
+                raise NotImplementedError("a gate on the shared expert goes with SwiGLU")
+            hy.act_cols(U[:, c:c + n], A[:, oc:oc + on], "relu2")
+        else:
+            hy.swiglu_cols(U[:, c:c + n], U[:, L.sg_col[0]:L.sg_col[0] + 1] if L.sg_col is not None else None, A[:, oc:oc + on])
+
     def _feed_forward(self, L, U, A):
         spec = L.spec
         c, n = L.ff_col
         oc, on = L.ff_out_col
-        if spec.ff_kind == "moe" and spec.route == "softmax_all":
+        if spec.ff_kind == "moe" and spec.route in ("softmax_all", "sigmoid_all"):
             rc, E = L.router_col
             self_w = torch.empty(U.shape[0], dtype=torch.float32, device=U.device) if spec.identity_experts else None
             hy.moe_route_all(U[:, rc:rc + E], L.router_bias, spec.experts, spec.top, spec.route_scale, gu=U[:, c:c + n], ff=spec.ff,
-                             act=A[:, oc:oc + on], self_w=self_w, groups=spec.route_groups, keep=spec.route_keep)
+                             act=A[:, oc:oc + on], self_w=self_w, groups=spec.route_groups, keep=spec.route_keep,
+                             sigmoid=spec.route == "sigmoid_all", group_score=spec.group_score, relu2=spec.ff_act == "relu2")
             return self_w
         if spec.ff_kind == "moe":
             rc, E = L.router_col
             hy.moe_route(U[:, rc:rc + E], L.router_bias, spec.top, gu=U[:, c:c + n], ff=spec.ff, act=A[:, oc:oc + on],
                          sigmoid=spec.route == "sigmoid", weight_input=spec.weight_input)
         elif spec.ff_act == "swiglu":
-            hy.swiglu_cols(U[:, c:c + n], None, A[:, oc:oc + on])
+            hy.swiglu_cols(U[:, c:c + n], None, A[:, oc:oc + on], spec.ff_alpha, spec.ff_limit, spec.ff_up_shift)
         else:
             hy.act_cols(U[:, c:c + n], A[:, oc:oc + on], spec.ff_act)
         return None
