@@ -1,7 +1,8 @@
 """Serving throughput of the hybrid step engine (Nezavik) beside the paged-KV transformer engine (Qwen2) at equal size,
 plus each new kernel against its roofline and against the like kernel of the transformer path; with ``--serve-model vilosun``
 the Vilosun family beside Nezavik (same engine) at equal size, and the kernels it adds beside Nezavik's like kernels; with
-``--serve-model damilix`` the Damilix family beside Vilosun in the same way, ``--serve-model lukarax`` the Lukarax family and ``--serve-model lopovik`` the Lopovik family beside Damilix.
+``--serve-model damilix`` the Damilix family beside Vilosun in the same way, ``--serve-model lukarax`` the Lukarax family and ``--serve-model lopovik`` the Lopovik family beside Damilix,
+``--serve-model lapilorn`` the Lapilorn family beside Lukarax.
 
 Run through ``python bench.py --serve-bench`` (one GPU).  Random weights, synthetic token ids.  End-to-end numbers go
 through the engines' public ``generate`` (two runs that differ by `new` generated tokens: the difference is `new` decode steps,
@@ -902,10 +903,202 @@ def kernels_lopovik(width=2048, batch=16, prompt_len=2048, decode_batch=256, ctx
     return out
 
 
+def lapilorn_config(width: int, n_layers: int, vocab: int, experts: int = 16, top: int = 2):
+    """Heads of 128 columns, four query heads per key/value head; layer pattern attention / lightning / attention reading the pages of
+    the layer two before / lightning; the clamped dense feed-forward on attention layers, squared-ReLU experts in four groups plus a
+    shared one on the others, each with as many active weights as a dense 4 x width feed-forward of two matrices."""
+    from nanorlhf_b200.models.lapilorn import LapilornConfig
+    H = width // 128
+    at = {"type": "attention", "mlp": {"kind": "dense", "ff": (8 * width // 3 + 127) // 128 * 128, "limit": 7.0},
+          "mixer": {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+                    "rot": {"base": 5e5, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}}}}
+    ff = (4 * width // (top + 1) + 127) // 128 * 128
+    li = {"type": "lightning", "mlp": {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": ff},
+                                       "router": {"experts": experts, "top": top, "scale": 2.0, "groups": {"count": 4, "keep": 2}}},
+          "mixer": {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-1 - 8.0 * (h + 1) / H) for h in range(H)]}}
+    layers = []
+    for i in range(n_layers):
+        layer = json.loads(json.dumps((at, li)[i % 2]))
+        if i % 4 == 2:
+            layer["mixer"]["kv_from"] = i - 2
+        layers.append(layer)
+    return LapilornConfig.from_dict({"architecture": "Lapilorn", "layers": layers, "norm": {"eps": 1e-6}, "vocab": vocab, "width": width})
+
+
+def end_to_end_lapilorn(width, n_layers, batch, prompt_len, new=128, vocab=32768):
+    """Lapilorn beside Lukarax (the closest family: capped rotated attention, borrowed pages, a recurrent matrix memory, grouped experts)
+    at equal width and depth."""
+    from nanorlhf_b200.models.lapilorn import LapilornForCausalLM
+    from nanorlhf_b200.models.lukarax import LukaraxForCausalLM
+    from nanorlhf_b200.sampler.hybrid_sampler import HybridSampler
+    dev = torch.device("cuda:0")
+    g = torch.Generator().manual_seed(0)
+    prompts = torch.randint(0, vocab - 2, (batch, prompt_len), generator=g).tolist()
+    res = {"width": width, "layers": n_layers, "batch": batch, "prompt_len": prompt_len, "new_tokens": new}
+    for name, make in (("lapilorn", lambda: LapilornForCausalLM.from_config(lapilorn_config(width, n_layers, vocab), torch.bfloat16, dev, seed=0)),
+                       ("lukarax", lambda: LukaraxForCausalLM.from_config(lukarax_config(width, n_layers, vocab), torch.bfloat16, dev, seed=0))):
+        model = make()
+        eng = HybridSampler(model, dtype="bf16", max_num_seqs=batch, prefill_token_budget=16384)
+        pre, step = _gen_times(lambda p, mt: eng.generate(p, 1, 1.0, 1.0, mt, None, vocab - 1, 1), prompts, new)
+        res[name] = {"params_m": round(sum(p.numel() for p in model.parameters()) / 1e6, 1),
+                     "prefill_tok_s": round(batch * prompt_len / pre), "decode_tok_s": round(batch / step),
+                     "decode_ms_per_step": round(step * 1e3, 3)}
+        eng.release()
+        del eng, model
+        torch.cuda.empty_cache()
+    return res
+
+
+def kernels_lapilorn(width=2048, batch=16, prompt_len=2048, decode_batch=256, ctx=2048, experts=16, top=2):
+    """The kernels Lapilorn adds to the step engine or extends, each beside the like kernel of the Lukarax / Lopovik / Damilix paths."""
+    from nanorlhf_b200 import _C
+    from nanorlhf_b200.ops import hybrid as hy
+    from nanorlhf_b200.sampler.hybrid_sampler import StepPlan
+    hbm, flops_peak, which = _peaks()
+    dev = torch.device("cuda:0")
+    out = {"roofline": which, "width": width}
+    H, Hkv, D = width // 128, max(1, width // 512), 128
+    bf = torch.bfloat16
+    n = H * D
+
+    def plan_for(B, n_new, n_old):
+        s = _C.StepScheduler((n_old + n_new + 15) // 16 * B + 8, 16, B)
+        sids = [s.open() for _ in range(B)]
+        if n_old:
+            s.plan(sids, [n_old] * B)
+        data, E, T, MB = s.plan(sids, [n_new] * B)
+        return StepPlan(torch.from_numpy(data).to(dev), E, T, MB), s
+
+    def report(name, sec, bytes_, flops=0.0):
+        floor = max(bytes_ / hbm, flops / flops_peak)
+        out[name] = {"us": round(sec * 1e6, 1), "gb_s": round(bytes_ / sec / 1e9, 1), "tflop_s": round(flops / sec / 1e12, 2),
+                     "roofline_frac": round(floor / sec, 3)}
+
+    for phase, B, n_new, n_old in (("prefill", batch, prompt_len, 0), ("decode", decode_batch, 1, ctx - 1)):
+        plan, sched = plan_for(B, n_new, n_old)
+        T = plan.T
+        tm = _time_graphed if phase == "decode" else _time
+        f32 = dict(dtype=torch.float32, device=dev)
+        plan.tokens.copy_(torch.randint(0, 32000, (T,), dtype=torch.int32, device=dev))
+        emb = torch.randn(32768, width, device=dev).bfloat16()
+        # -- layer boundary: residual add, one norm, weighted expert rows; beside two norms with a token shift and plain rows
+        x, o, xn = torch.randn(T, width, **f32), torch.randn(T, width, **f32), torch.empty(T, width, **f32)
+        h1, h2 = torch.empty(T, width, dtype=bf, device=dev), torch.empty(T, width, dtype=bf, device=dev)
+        w1, mu = torch.ones(width, **f32), torch.full((width,), 0.3, **f32)
+        state, carry = torch.zeros(B, width, **f32), torch.empty(B, width, **f32)
+        y, slot_of = torch.randn(T * top, width, **f32), torch.randperm(T * top, device=dev).int()
+        wk = torch.rand(T, top, **f32)
+        one = dict(x_in=x, o=o, w1=w1, x_out=xn, h1=h1)
+        two = dict(one, w2=w1, mu=mu, h2=h2, state=state, carry=carry, commit=carry.clone(), commit_state=torch.zeros(B, width, **f32))
+        sec = tm(lambda: hy.parallel_boundary(plan, emb, 1e-6, **one))
+        report(f"{phase}.parallel_boundary(one norm)", sec, T * width * (4.0 * 3 + 2))
+        sec = tm(lambda: hy.parallel_boundary(plan, emb, 1e-6, y=y, slot_of=slot_of, wts=wk, **one))
+        report(f"{phase}.parallel_boundary(one norm, {top} weighted expert rows)", sec, T * width * (4.0 * (3 + top) + 2) + T * top * 8.0)
+        sec = tm(lambda: hy.parallel_boundary(plan, emb, 1e-6, **two))
+        report(f"{phase}.lopovik.parallel_boundary", sec, T * width * (4.0 * 3 + 2 * 2) + B * width * 16.0)
+        sec = tm(lambda: hy.parallel_boundary(plan, emb, 1e-6, y=y, slot_of=slot_of, **two))
+        report(f"{phase}.lopovik.parallel_boundary(+ {top} expert rows)", sec, T * width * (4.0 * (3 + top) + 2 * 2) + B * width * 16.0)
+        del x, o, xn, h2, y, two
+        # -- write side of the attention, with its own keys and reading another layer's
+        n_pages = sched.num_free_blocks() + plan.max_blocks * B + 8
+        nk = Hkv * D
+        q, k_, v_ = torch.randn(T, n, **f32), torch.randn(T, nk, **f32), torch.randn(T, nk, **f32)
+        kc, vc = (torch.randn(n_pages, Hkv, 16, D, device=dev).bfloat16() for _ in range(2))
+        fr, mult = hy.rotary_frequencies(64, 5e5, {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096})
+        freq = torch.tensor(fr, dtype=torch.float64, device=dev)
+        ff_, fm = hy.rotary_frequencies(64, 1e6, {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0})
+        freq2 = torch.tensor(ff_, dtype=torch.float64, device=dev)
+        sec = tm(lambda: hy.rot_kv_write(q, None, k_, None, v_, freq, 64, mult, True, False, None, None, 1e-6, plan, kc, vc))
+        report(f"{phase}.rot_kv_write(q, k, v)", sec, T * (n * 8.0 + nk * (8.0 + 4.0)))
+        sec = tm(lambda: hy.rot_kv_write(q, None, None, None, None, freq, 64, mult, True, False, None, None, 1e-6, plan, kc, vc))
+        report(f"{phase}.rot_kv_write(q)", sec, T * n * 8.0)
+        qb, kb = torch.randn(n, **f32), torch.randn(nk, **f32)
+        sec = tm(lambda: hy.rot_kv_write(q, qb, k_, kb, None, freq2, 64, fm, False, True, None, None, 1e-6, plan, kc, vc))
+        report(f"{phase}.lukarax.rot_kv_write(values = keys)", sec, T * (n * 8.0 + nk * (4.0 + 4.0)))
+        # -- causal attention: cap and gate per column; the same without the gate, with the cap alone, and plain
+        q.normal_()
+        ao, gate = torch.empty(T, n, dtype=bf, device=dev), torch.randn(T, n, **f32)
+        ta = (lambda f: _time(f, iters=3, warm=1)) if phase == "prefill" else (lambda f: _time(f, iters=20, warm=5))
+        keys = (sum(p + 1 for p in range(n_new)) if phase == "prefill" else ctx) * B
+        byt = (T * n * 6.0 + T * 2 * nk * 2.0) if phase == "prefill" else (keys * 2 * nk * 2.0 + T * n * 6.0)
+        fl = 4.0 * keys * n
+        sec = ta(lambda: hy.window_attention(q, kc, vc, plan, 1 << 30, D ** -0.5, 1.0, ao, gate=gate, softcap=50.0))
+        report(f"{phase}.attention(causal, cap, column gate)", sec, byt + T * n * 4.0, flops=fl)
+        sec = ta(lambda: hy.window_attention(q, kc, vc, plan, 1 << 30, D ** -0.5, 1.0, ao, softcap=50.0))
+        report(f"{phase}.lukarax.attention(causal, cap)", sec, byt, flops=fl)
+        sec = ta(lambda: hy.window_attention(q, kc, vc, plan, 1 << 30, D ** -0.5, 1.0, ao))
+        report(f"{phase}.nezavik.attention(causal)", sec, byt, flops=fl)
+        del kc, vc, q
+        # -- constant-decay linear attention vs gated linear attention and the matrix memory (same state size), and the read-out norms
+        U = torch.randn(T, 4 * n, **f32) * 0.5
+        pows, st = hy.decay_powers([1.0 - 2.0 ** (-1 - 8.0 * (h + 1) / H) for h in range(H)], dev), torch.zeros(B, H, D, D, **f32)
+        ol = torch.empty(T, n, **f32)
+        ts = lambda f: _time(f, iters=5, warm=2)
+        sec = ts(lambda: hy.lightning_scan(U, 0, n, 2 * n, pows, st, ol, plan, True))
+        report(f"{phase}.lightning_scan", sec, B * H * D * D * 8.0 + T * n * 16.0, flops=4.0 * T * n * D)
+        if phase == "prefill":
+            sec = ts(lambda: hy.lightning_scan(U, 0, n, 2 * n, pows, st, ol, plan, False))
+            report(f"{phase}.lightning_scan(token by token)", sec, B * H * D * D * 8.0 + T * n * 16.0, flops=4.0 * T * n * D)
+        decay = torch.rand(T, n, **f32) * 0.1 + 0.9
+        sec = ts(lambda: hy.delta_scan(U[:, :3 * n], n, 2 * n, None, decay, st, ol, plan, H, True))
+        report(f"{phase}.damilix.gla_scan", sec, B * H * D * D * 8.0 + T * n * 20.0, flops=4.0 * T * n * D)
+        del decay
+        sm, mst = torch.zeros(B, H, D, D + 8, **f32), torch.zeros(B, H, **f32)
+        om, mo, ib = torch.empty(T, H * (D + 1), **f32), torch.empty(T, H, **f32), torch.zeros(H, **f32)
+        sec = ts(lambda: hy.mlstm_scan(U, 0, n, 2 * n, 3 * n, 3 * n + H, ib, ib, 15.0, D ** -0.5, sm, mst, om, mo, plan))
+        report(f"{phase}.lukarax.mlstm_scan", sec, B * H * D * D * 8.0 + T * n * 16.0, flops=4.0 * T * n * D)
+        nw = torch.ones(n, **f32)
+        sec = tm(lambda: hy.gated_part_rmsnorm(ol, gate, nw, n, "sigmoid", False, 1e-6, 1.0, ao))
+        report(f"{phase}.gated_part_rmsnorm(all heads together)", sec, T * n * 10.0)
+        sec = tm(lambda: hy.mlstm_out(om, mo, gate, nw, 1e-6, 1.0, ao, H))
+        report(f"{phase}.lukarax.mlstm_out", sec, T * n * 10.0)
+        del U, om, ol, gate, ao, st, sm
+        # -- feed-forwards: clamped unit vs SwiGLU; squared ReLU of the shared expert; sigmoid routing with group sums vs softmax with groups
+        fd = (8 * width // 3 + 127) // 128 * 128
+        gu, act = torch.randn(T, 2 * fd, **f32), torch.empty(T, fd, dtype=bf, device=dev)
+        sec = tm(lambda: hy.swiglu_cols(gu, None, act, 1.702, 7.0, 1.0))
+        report(f"{phase}.swiglu_cols(clamped)", sec, T * fd * 10.0)
+        sec = tm(lambda: hy.swiglu_cols(gu, None, act))
+        report(f"{phase}.damilix.swiglu_cols", sec, T * fd * 10.0)
+        sec = tm(lambda: hy.act_cols(gu[:, :fd], act, "relu2"))
+        report(f"{phase}.act_cols(relu2)", sec, T * fd * 6.0)
+        del gu, act
+        z, corr = torch.randn(T, experts, **f32), torch.randn(experts, **f32) * 0.02
+        ids, wts = torch.empty(T, top, dtype=torch.int32, device=dev), torch.empty(T, top, **f32)
+        rb = T * (experts * 4.0 + top * 8.0)
+        sec = tm(lambda: hy.moe_route_all(z, corr, experts, top, 2.0, ids=ids, wts=wts, groups=4, keep=2))
+        report(f"{phase}.lukarax.moe_route_all(4 groups)", sec, rb)
+        sec = tm(lambda: hy.moe_route_all(z, corr, experts, top, 2.0, ids=ids, wts=wts, groups=4, keep=2, sigmoid=True, group_score="top2"))
+        report(f"{phase}.moe_route_all(sigmoid, 4 groups by their two best)", sec, rb)
+        ff = (4 * width // (top + 1) + 127) // 128 * 128
+        wu = (torch.randn(experts * ff, width, device=dev) * width ** -0.5).bfloat16()
+        wd = (torch.randn(experts * width, ff, device=dev) * ff ** -0.5).bfloat16()
+        hit = min(experts, T * top)
+        sec = tm(lambda: hy.moe_grouped_ffn(h1, ids, wts, wu, wd, experts, ff, None, relu2=True))
+        report(f"{phase}.moe_grouped_ffn(squared ReLU, rows out)", sec, hit * 2.0 * ff * width * 2.0 + T * width * (2.0 + 4.0 * top), flops=4.0 * T * top * width * ff)
+        wg, res = (torch.randn(experts * 2 * ff, width, device=dev) * width ** -0.5).bfloat16(), torch.empty(T, width, **f32)
+        sec = tm(lambda: hy.moe_grouped_ffn(h1, ids, wts, wg, wd, experts, ff, res, fused_act=True))
+        report(f"{phase}.lukarax.moe_grouped_ffn(SwiGLU, combined)", sec, hit * 3.0 * ff * width * 2.0 + T * width * 6.0, flops=6.0 * T * top * width * ff)
+        del wu, wd, wg
+    return out
+
+
 def main(quick: bool = False, small: bool = False, model: str = "nezavik"):
     from nanorlhf_b200.ops import native
     global SMALL
     native.load()
+    if model == "lapilorn":
+        SMALL = small
+        if small:
+            print(json.dumps({"bench": "serve-lapilorn-small",
+                              "kernels": kernels_lapilorn(width=1024, batch=8, prompt_len=1024, decode_batch=64, ctx=1024)}))
+            return None
+        res = {"bench": "serve-lapilorn", "kernels": kernels_lapilorn(), "end_to_end": []}
+        for width, layers, batch, plen in ((1024, 8, 32, 1024), (2048, 8, 16, 2048)) if not quick else ((1024, 4, 8, 512),):
+            res["end_to_end"].append(end_to_end_lapilorn(width, layers, batch, plen))
+        res["gpu_launches"] = native.launches()
+        print(json.dumps(res))
+        return res
     if model == "lopovik":
         SMALL = small
         if small:
@@ -968,4 +1161,4 @@ def main(quick: bool = False, small: bool = False, model: str = "nezavik"):
 
 if __name__ == "__main__":
     main(quick="--quick" in sys.argv, small="--small" in sys.argv,
-         model="lopovik" if "--lopovik" in sys.argv else "lukarax" if "--lukarax" in sys.argv else "damilix" if "--damilix" in sys.argv else "vilosun" if "--vilosun" in sys.argv else "nezavik")
+         model="lapilorn" if "--lapilorn" in sys.argv else "lopovik" if "--lopovik" in sys.argv else "lukarax" if "--lukarax" in sys.argv else "damilix" if "--damilix" in sys.argv else "vilosun" if "--vilosun" in sys.argv else "nezavik")
